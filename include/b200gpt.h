@@ -377,6 +377,7 @@ typedef struct b200_rms_rows_seg {
   const int64_t* out_rows;
   int64_t ld_in, ld_out;
   int d, plus_one;
+  int center;   /* the row minus its mean is normed: a layer norm without bias */
 } b200_rms_rows_seg;
 int b200_rms_rows(const b200_rms_rows_seg* segs, int n_segs, int64_t rows, float eps, int in_dtype, int out_dtype, b200_stream_t stream);
 /* x[row] += y[row] / sqrt(mean(y[row]^2) + eps) * (1 + weight); act[row] = dtype(x[row]) */
@@ -487,12 +488,17 @@ typedef struct b200_sandwich_args {
   const void* post_w; const float* extra; const void* pre_w;
   float* x; void* act;
   int64_t rows; int d; float eps; int dtype;
+  int pre_center;   /* act is the norm of x minus its mean (a layer norm without bias) */
+  void* cast;       /* optional: dtype(x) */
 } b200_sandwich_args;
 int b200_sandwich_residual(const b200_sandwich_args* args, b200_stream_t stream);
 /* in place; kind 0 exact gelu (erf), 1 tanh gelu, 2 silu, 3 relu^2 */
 int b200_activation(void* x, int64_t n, int kind, int dtype, b200_stream_t stream);
 /* out[r, c] = act(in[r, c]) * in[r, ff + c] for in (rows, 2 ff) */
 int b200_glu(const void* in, void* out, int64_t rows, int ff, int kind, int dtype, b200_stream_t stream);
+/* out[r, c] = act(z[r, c]) * table[tokens[r], off + c] for c < cols; act as in b200_activation; table (vocab, ld_table) */
+int b200_token_gate(const void* z, int64_t ldz, const int32_t* tokens, const void* table, int64_t ld_table, int64_t off, int vocab, void* out,
+                    int64_t rows, int cols, int kind, int dtype, b200_stream_t stream);
 /* in place: xIELU with its two raw parameters params[0..1] (in `dtype`): z > 0: softplus(p) z^2 + z / 2, else (1/2 + softplus(q)) (exp(z) - 1 - z) + z / 2 */
 int b200_xielu(void* x, int64_t n, const void* params, int dtype, b200_stream_t stream);
 /* in (rows, 2 ff) = [gate | up] -> out (rows, ff) = g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit) */
@@ -574,13 +580,48 @@ typedef struct b200_window_attn_args {
   const void* dist_r1; const void* dist_r2;
   /* optional: the output is multiplied by sigmoid(gate[row, h]) (gate_mode 1) or sigmoid(gate[row, h * dv + c]) (gate_mode 2); rows ldg apart */
   const void* gate; int64_t ldg; int gate_mode;
+  /* optional (0: none): positions j < keep stay visible whatever the window; score <- softcap * tanh(score / softcap) after the scale.
+   * The rings then hold keep + ring rows per slot: position p in row p when p < keep, else in row keep + (p - keep) % ring. */
+  int keep; float softcap;
 } b200_window_attn_args;
 int b200_window_attn(const b200_window_attn_args* args, b200_stream_t stream);
+/* The tensor-core tiles of b200_attn_prefill_window for the same description, without distance bias and without touching the rings:
+ * bf16, dk and dv multiples of 8 up to 128 (they may differ), every sequence at position 0, leading dimensions of q, k, v multiples of 8
+ * elements, q / k / v / seqs 16-byte aligned. */
+int b200_window_attn_tiles(const b200_window_attn_args* args, b200_stream_t stream);
 /* test knob: non-zero keeps single-row steps on the tiled kernel; returns the previous setting */
 int b200_window_attn_tune(int force_tiled_kernel);
 /* the step's rows among each sequence's last `ring` positions go to their ring rows (call after b200_window_attn) */
 int b200_ring_store(const void* k, int64_t ldk, const void* v, int64_t ldv, void* k_ring, void* v_ring, int ring, int kcols, int vcols,
                     const int32_t* seqs, const int32_t* row_seq, int64_t rows, int dtype, b200_stream_t stream);
+
+
+/* b200_ring_store with `keep` first rows per slot that are never replaced (see b200_window_attn_args) */
+int b200_ring_store_keep(const void* k, int64_t ldk, const void* v, int64_t ldv, void* k_ring, void* v_ring, int ring, int keep, int kcols, int vcols,
+                         const int32_t* seqs, const int32_t* row_seq, int64_t rows, int dtype, b200_stream_t stream);
+
+/* Decaying linear attention over fp32 states, one dk x dv matrix per (slot, head), stored [head][dk][dv]: per token S <- diag(g) S + k v^T,
+ * o = S^T q.  q, k (rows, heads * dk) and v (rows, heads * dv) are projections in `dtype`, each through silu when act is 1, q then times
+ * q_scale.  Decays: head_decay[heads], fixed -- or decay_in (rows, heads * dk) fp32 raw with decay_bias (heads * dk, `dtype`) and tau,
+ * g = sigmoid(decay_in + decay_bias)^(1 / tau) (decay_in is scratch: its rows may be overwritten).  A sequence at position 0 starts from
+ * S = 0.  Long prompts run in pieces side by side, for which the workspace holds a state per piece. */
+typedef struct b200_linear_attn_args {
+  const void* q; const void* k; const void* v;
+  int64_t ldq, ldk, ldv;
+  int act; float q_scale;
+  float* decay_in; int64_t ld_decay; const void* decay_bias; float tau;
+  const float* head_decay;
+  float* state; int64_t state_slot_stride;
+  float* out; int64_t ldo;
+  const int32_t* seqs; int n_seqs;
+  int64_t rows; int max_rows;       /* rows of the step; of its longest sequence */
+  int heads, dk, dv, dtype;
+  void* workspace; size_t workspace_bytes;
+} b200_linear_attn_args;
+size_t b200_linear_attn_workspace_bytes(int64_t rows, int max_rows, int n_seqs, int heads, int dk, int dv);
+int b200_linear_attn(const b200_linear_attn_args* args, b200_stream_t stream);
+/* test and tuning knob: tokens per piece of a prompt (0: chosen by size); returns the previous setting */
+int b200_linear_attn_tune(int piece);
 
 
 /* ---- grouped norms with an average over depth, per-head rotation, attention whose scores mix over the heads ------------------ */
@@ -598,12 +639,14 @@ int b200_depth_residual(const b200_depth_residual_args* args, b200_stream_t stre
 /* One group of heads of b200_head_rope: head h of a row is `dim` numbers at in + row * ld_in + h * in_stride and goes to
  * out + out_rows[row] * ld_out + h * out_stride (out_rows NULL: the row itself; a row < 0 is skipped; in place allowed).  norm_w
  * (dim numbers, NULL: no norm) is the weight of an RMS norm over the head; dimensions [rot_off, rot_off + rot_dims) turn by
- * position * freq[i] (fp32), pair i = (2 i, 2 i + 1) when interleaved, else (i, i + rot_dims / 2), cos and sin times mag. */
+ * position * freq[i] (fp32, or fp64 with freq_f64), pair i = (2 i, 2 i + 1) when interleaved, else (i, i + rot_dims / 2), cos and sin
+ * times mag.  norm_all: one norm over all heads of the row at once (in_stride = dim), norm_w then holds heads * dim numbers. */
 typedef struct b200_head_rope_seg {
-  const void* in; void* out; const void* norm_w; const float* freq; const int64_t* out_rows;
+  const void* in; void* out; const void* norm_w; const void* freq; const int64_t* out_rows;
   int64_t ld_in, ld_out;
   int heads, dim, in_stride, out_stride, rot_off, rot_dims, interleaved;
   float mag;
+  int norm_all, freq_f64;
 } b200_head_rope_seg;
 int b200_head_rope(const b200_head_rope_seg* segs, int n_segs, const int32_t* row_pos, int64_t rows, float eps, int dtype, b200_stream_t stream);
 /* Causal attention over cached keys and values in which the heads' scores are mixed before the softmax:

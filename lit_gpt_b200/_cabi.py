@@ -76,7 +76,7 @@ class QGemmArgs(ctypes.Structure):
 
 class RmsRowsSeg(ctypes.Structure):  # mirrors b200_rms_rows_seg
     _fields_ = [("inp", c_void_p), ("weight", c_void_p), ("out", c_void_p), ("in_rows", c_void_p), ("out_rows", c_void_p),
-                ("ld_in", c_int64), ("ld_out", c_int64), ("d", c_int), ("plus_one", c_int)]
+                ("ld_in", c_int64), ("ld_out", c_int64), ("d", c_int), ("plus_one", c_int), ("center", c_int)]
 
 
 class LatentPrefillArgs(ctypes.Structure):  # mirrors b200_latent_prefill_args
@@ -104,7 +104,7 @@ class DepthResidualArgs(ctypes.Structure):  # mirrors b200_depth_residual_args
 class HeadRopeSeg(ctypes.Structure):  # mirrors b200_head_rope_seg
     _fields_ = [("inp", c_void_p), ("out", c_void_p), ("norm_w", c_void_p), ("freq", c_void_p), ("out_rows", c_void_p), ("ld_in", c_int64),
                 ("ld_out", c_int64), ("heads", c_int), ("dim", c_int), ("in_stride", c_int), ("out_stride", c_int), ("rot_off", c_int),
-                ("rot_dims", c_int), ("interleaved", c_int), ("mag", c_float)]
+                ("rot_dims", c_int), ("interleaved", c_int), ("mag", c_float), ("norm_all", c_int), ("freq_f64", c_int)]
 
 
 class TalkAttnArgs(ctypes.Structure):  # mirrors b200_talk_attn_args
@@ -116,7 +116,8 @@ class TalkAttnArgs(ctypes.Structure):  # mirrors b200_talk_attn_args
 
 class SandwichArgs(ctypes.Structure):  # mirrors b200_sandwich_args
     _fields_ = [("y0", c_void_p), ("w0", c_void_p), ("y1", c_void_p), ("w1", c_void_p), ("post_w", c_void_p), ("extra", c_void_p),
-                ("pre_w", c_void_p), ("x", c_void_p), ("act", c_void_p), ("rows", c_int64), ("d", c_int), ("eps", c_float), ("dtype", c_int)]
+                ("pre_w", c_void_p), ("x", c_void_p), ("act", c_void_p), ("rows", c_int64), ("d", c_int), ("eps", c_float), ("dtype", c_int),
+                ("pre_center", c_int), ("cast", c_void_p)]
 
 
 class ConvGroup(ctypes.Structure):  # mirrors b200_conv_group
@@ -138,7 +139,15 @@ class WindowAttnArgs(ctypes.Structure):  # mirrors b200_window_attn_args
                 ("ldo", c_int64), ("k_ring", c_void_p), ("v_ring", c_void_p), ("sink", c_void_p), ("seqs", c_void_p), ("n_seqs", c_int),
                 ("max_q_len", c_int), ("ring", c_int), ("n_head", c_int), ("n_kv_head", c_int), ("dk", c_int), ("dv", c_int), ("window", c_int),
                 ("scale", c_float), ("dtype", c_int), ("row_seq", c_void_p), ("rows", c_int64), ("dist_r1", c_void_p), ("dist_r2", c_void_p),
-                ("gate", c_void_p), ("ldg", c_int64), ("gate_mode", c_int)]
+                ("gate", c_void_p), ("ldg", c_int64), ("gate_mode", c_int), ("keep", c_int), ("softcap", c_float)]
+
+
+class LinearAttnArgs(ctypes.Structure):  # mirrors b200_linear_attn_args
+    _fields_ = [("q", c_void_p), ("k", c_void_p), ("v", c_void_p), ("ldq", c_int64), ("ldk", c_int64), ("ldv", c_int64), ("act", c_int),
+                ("q_scale", c_float), ("decay_in", c_void_p), ("ld_decay", c_int64), ("decay_bias", c_void_p), ("tau", c_float), ("head_decay", c_void_p),
+                ("state", c_void_p), ("state_slot_stride", c_int64), ("out", c_void_p), ("ldo", c_int64), ("seqs", c_void_p), ("n_seqs", c_int),
+                ("rows", c_int64), ("max_rows", c_int), ("heads", c_int), ("dk", c_int), ("dv", c_int), ("dtype", c_int), ("workspace", c_void_p),
+                ("workspace_bytes", c_size_t)]
 
 
 class ScaledResidualArgs(ctypes.Structure):  # mirrors b200_scaled_residual_args
@@ -153,7 +162,7 @@ ACT_GELU, ACT_GELU_TANH, ACT_SILU, ACT_RELU2 = 0, 1, 2, 3
 # Entry points of the sources every model needs (library state, norms, sampling) and of the fp32-residual / latent-attention /
 # expert kernels: `load_core()` can serve them from a library built from those sources alone.
 _CORE_SOURCES = ("api.cu", "norm.cu", "sample.cu", "resid.cu", "latent.cu", "moe.cu", "attn_prefill.cu", "shortconv.cu", "delta.cu", "window_attn.cu",
-                 "depth.cu", "rope.cu", "talk_attn.cu")
+                 "linear_attn.cu", "depth.cu", "rope.cu", "talk_attn.cu")
 _CORE_SIGNATURES = {
     "b200_embed_pos": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_void_p]),
     "b200_rms_rows": (c_int, [ctypes.POINTER(RmsRowsSeg), c_int, c_int64, c_float, c_int, c_int, c_void_p]),
@@ -191,6 +200,13 @@ _CORE_SIGNATURES = {
                                      c_void_p]),
     "b200_window_attn": (c_int, [ctypes.POINTER(WindowAttnArgs), c_void_p]),
     "b200_window_attn_tune": (c_int, [c_int]),
+    "b200_window_attn_tiles": (c_int, [ctypes.POINTER(WindowAttnArgs), c_void_p]),
+    "b200_ring_store_keep": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int64,
+                                     c_int, c_void_p]),
+    "b200_linear_attn_workspace_bytes": (c_size_t, [c_int64, c_int, c_int, c_int, c_int, c_int]),
+    "b200_linear_attn": (c_int, [ctypes.POINTER(LinearAttnArgs), c_void_p]),
+    "b200_linear_attn_tune": (c_int, [c_int]),
+    "b200_token_gate": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int64, c_int, c_void_p, c_int64, c_int, c_int, c_int, c_void_p]),
     "b200_depth_residual": (c_int, [ctypes.POINTER(DepthResidualArgs), c_void_p]),
     "b200_head_rope": (c_int, [ctypes.POINTER(HeadRopeSeg), c_int, c_void_p, c_int64, c_float, c_int, c_void_p]),
     "b200_attn_prefill_mixed_plane_floats": (c_size_t, [c_int, c_int, c_int64]),

@@ -603,7 +603,9 @@ class FizadraConfig:
 class GatedWindowSpec:
     """Sliding-window attention with a sigmoid output gate: optional biases on the q, k, v projections, optional rotary positions
     (half-split pairs) on q and k, an optional distance bias (score -= r1_h ln(1 + r2_h (i - j)), two learned numbers per head), and
-    a gate per output number ("element") or per head ("head") projected from the mixer's input."""
+    a gate per output number ("element") or per head ("head") projected from the mixer's input.  Also optional: an RMS norm with weights
+    over all query heads at once, and one over all key heads, before the rotation (`qk_norm`); a soft cap on the scaled scores; the first
+    `keep` positions of a sequence staying visible whatever the window; a learned logit per head in the softmax denominator (`sink`)."""
 
     heads: int
     kv_heads: int
@@ -615,6 +617,10 @@ class GatedWindowSpec:
     bias: bool = False
     distance: bool = False
     gate: Optional[str] = "element"
+    qk_norm: bool = False
+    softcap: float = 0.0           # 0: none
+    keep: int = 0                  # first positions that never leave the window
+    sink: bool = False
 
 
 @dataclass
@@ -729,11 +735,116 @@ class NulezenConfig:
             return cls.from_dict(json.load(fp))
 
 
+@dataclass
+class LinearMixerSpec:
+    """Linear attention with decaying states: S <- diag(g) S + k v^T, o = S^T q per head.  `decay` set: one fixed decay per head, q, k, v
+    through silu, the heads normed together, a sigmoid output gate.  Else a decay per head and key channel, sigmoid(z)^(1 / tau) of a
+    low-rank projection (inner size `decay_rank`), q times dim^-1/2, each head normed alone, a silu output gate."""
+
+    heads: int
+    dim: int
+    vdim: int
+    decay: Optional[List[float]] = None
+    tau: float = 1.0
+    decay_rank: int = 0            # read from the weights' shapes
+
+
+@dataclass
+class ClampedGLUSpec:
+    """Dense feed-forward W_down (g sigmoid(alpha g) (u + 1)), g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit)."""
+
+    ff: int
+    limit: float
+    alpha: float = 1.702
+
+
+@dataclass
+class VotavikLayerSpec:
+    type: str                      # "attention" | "gla" | "lightning"
+    mixer: Any                     # GatedWindowSpec | LinearMixerSpec
+    mlp: Optional[ClampedGLUSpec] = None
+
+
+@dataclass
+class VotavikConfig:
+    """Votavik: pre-normed blocks (layer norms without bias) over an fp32 residual stream, each ending with an input of its own from a
+    second embedding table, gated by the stream.  Mixers: sliding-window attention with kept first tokens, capped scores and a sink;
+    linear attention with a decay per channel ("gla") or a fixed one per head ("lightning"); feed-forwards gated and clamped, or none."""
+
+    name: str = "Votavik"
+    vocab_size: int = 0
+    n_embd: int = 0
+    norm_eps: float = 1e-5
+    side_dim: int = 0              # numbers per layer and token in the second embedding table
+    layers: List[VotavikLayerSpec] = field(default_factory=list)
+    block_size: int = 1 << 30      # constant-size state, no position table: positions are bounded by int32 only
+
+    def __post_init__(self) -> None:
+        self.padded_vocab_size = self.vocab_size
+        self.n_layer = len(self.layers)
+        if self.side_dim < 1:
+            raise ValueError("the per-layer token input needs a positive size")
+        for i, layer in enumerate(self.layers):
+            m = layer.mixer
+            if layer.type == "attention":
+                if m.heads < 1 or m.kv_heads < 1 or m.heads % m.kv_heads or m.window < 1 or m.dim < 1 or m.vdim < 1 or m.keep < 0 or m.softcap < 0:
+                    raise ValueError(f"layer {i}: bad attention shape")
+                if m.rot is not None and (m.rot.dims % 2 or m.rot.dims > m.dim):
+                    raise ValueError(f"layer {i}: rotary dimensions must be even and at most the head size")
+            elif layer.type in ("gla", "lightning"):
+                if m.heads < 1 or m.dim < 1 or m.vdim < 1:
+                    raise ValueError(f"layer {i}: bad linear-attention shape")
+                if layer.type == "lightning" and (m.decay is None or len(m.decay) != m.heads or not all(0.0 <= g <= 1.0 for g in m.decay)):
+                    raise ValueError(f"layer {i}: one decay in [0, 1] per head")
+                if layer.type == "gla" and not m.tau > 0.0:
+                    raise ValueError(f"layer {i}: tau must be positive")
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {layer.type!r}")
+            if layer.mlp is not None and (layer.mlp.ff < 1 or not layer.mlp.limit > 0.0):
+                raise ValueError(f"layer {i}: bad feed-forward (its limit must be positive)")
+
+    def schedule(self) -> List[Tuple[int, int]]:
+        """The layer runs in order: (layer index, state index)."""
+        return [(i, i) for i in range(self.n_layer)]
+
+    @classmethod
+    def from_dict(cls, js: Dict[str, Any]) -> "VotavikConfig":
+        layers = []
+        for i, entry in enumerate(js["layers"]):
+            mx, kind = entry["mixer"], entry["type"]
+            if kind == "attention":
+                rot, mask = mx.get("rot"), mx["mask"]
+                mixer: Any = GatedWindowSpec(
+                    heads=int(mx["heads"]), kv_heads=int(mx.get("kv_heads", mx["heads"])), dim=int(mx["dim"]), vdim=int(mx.get("vdim", mx["dim"])),
+                    window=int(mask["size"]), scale=float(mx["scale"]), rot=RotarySpec.from_dict(rot, interleaved=False) if rot and int(rot["dims"]) > 0 else None,
+                    gate="head", qk_norm=True, softcap=float(mx.get("softcap") or 0.0), keep=int(mask.get("keep_first") or 0), sink=True)
+            elif kind == "lightning":
+                mixer = LinearMixerSpec(heads=int(mx["heads"]), dim=int(mx["dim"]), vdim=int(mx.get("vdim", mx["dim"])), decay=[float(g) for g in mx["decay"]])
+            elif kind == "gla":
+                mixer = LinearMixerSpec(heads=int(mx["heads"]), dim=int(mx["dim"]), vdim=int(mx.get("vdim", mx["dim"])), tau=float(mx["tau"]))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer type {kind!r}")
+            mlp, ml = None, entry.get("mlp")
+            if ml is not None:
+                if ml.get("kind", "dense") != "dense":
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {ml.get('kind')!r}")
+                mlp = ClampedGLUSpec(ff=int(ml["ff"]), limit=float(ml["limit"]))
+            layers.append(VotavikLayerSpec(type=kind, mixer=mixer, mlp=mlp))
+        return cls(name=js.get("architecture", "Votavik"), vocab_size=int(js["vocab"]), n_embd=int(js["width"]), norm_eps=float(js["norm"]["eps"]),
+                   side_dim=int(js["token_side"]["dim"]), layers=layers)
+
+    @classmethod
+    def from_json(cls, path: Union[str, Path]) -> "VotavikConfig":
+        with open(path, encoding="utf-8") as fp:
+            return cls.from_dict(json.load(fp))
+
+
 # "architecture" value of config.json -> (configuration class, "module:class" of the model)
 architectures: Dict[str, Any] = {"Pomipel": (PomipelConfig, "lit_gpt_b200.pomipel:Pomipel"),
                                  "Lefalix": (LefalixConfig, "lit_gpt_b200.lefalix:Lefalix"),
                                  "Fizadra": (FizadraConfig, "lit_gpt_b200.fizadra:Fizadra"),
-                                 "Nulezen": (NulezenConfig, "lit_gpt_b200.nulezen:Nulezen")}
+                                 "Nulezen": (NulezenConfig, "lit_gpt_b200.nulezen:Nulezen"),
+                                 "Votavik": (VotavikConfig, "lit_gpt_b200.votavik:Votavik")}
 
 
 def load_config(checkpoint_dir: Union[str, Path], **kwargs: Any) -> Any:

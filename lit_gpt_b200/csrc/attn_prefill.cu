@@ -59,23 +59,29 @@ struct PfView {
   const __nv_bfloat16* dist_r1;
   const __nv_bfloat16* dist_r2;
   int bias_n;
+  // kernels instantiated with EX only: dk <= HS query / key and dv <= HV value numbers per head (multiples of 8; the tile's rest is
+  // zero), positions below `keep` that every later row sees besides its window, and a soft cap, cap * tanh(score / cap): cap_log2 =
+  // cap * log2(e), cap_in = 2 * scale / cap * log2(e) (0: no cap).
+  int dk, dv, keep;
+  float cap_log2, cap_in;
 };
 
 constexpr int kPfBiasTabMax = 8192;   // distances a CTA tabulates at most (32 KB)
 
-template <int HS, typename PosT, int HK2 = 0, int MODE = 0>
+template <int HS, typename PosT, int HK2 = 0, int MODE = 0, int HV = HS, bool EX = false>
 __global__ void __launch_bounds__(kPfThreads, 1)
 attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ kc, const __nv_bfloat16* __restrict__ vc,
                     const PosT* __restrict__ pos, __nv_bfloat16* __restrict__ y, int T, int n_head, int n_groups, int max_seq,
                     float scale_log2, PfView vw) {
   extern __shared__ __align__(128) uint8_t pf_smem_raw[];
   constexpr int CH = HS / 8;                         // 16-byte chunks per row
-  constexpr int QB = kPfBM * HS * 2, KB = kPfBN * HS * 2;
+  constexpr int CHV = HV / 8;
+  constexpr int QB = kPfBM * HS * 2, KB = kPfBN * HS * 2, VB = kPfBN * HV * 2;
   uint8_t* const sQ = pf_smem_raw;                   // [128][HS]
   uint8_t* const sK = sQ + QB;                       // [2][64][HS]
-  uint8_t* const sV = sK + 2 * KB;                   // [2][64][HS]
+  uint8_t* const sV = sK + 2 * KB;                   // [2][64][HV]
   constexpr int CH2 = HK2 / 8, KB2 = kPfBN * HK2 * 2;
-  uint8_t* const sQ2 = sV + 2 * KB;                  // [128][HK2]  the query columns that meet the shared key part
+  uint8_t* const sQ2 = sV + 2 * VB;                  // [128][HK2]  the query columns that meet the shared key part
   uint8_t* const sK2 = sQ2 + kPfBM * HK2 * 2;        // [2][64][HK2]
   float* const sTab = reinterpret_cast<float*>(sK2 + 2 * KB2);   // [bias_n] distance bias by distance, in units of the raw dot product
   __shared__ int s_maxpos[kPfThreads / 32];
@@ -121,8 +127,8 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   if constexpr (MODE != 2)
   for (int i = tid; i < kPfBM * CH; i += kPfThreads) {
     const int r = i / CH, c = i % CH;
-    const bool ok = r0 + r < T;
-    pf_cp16(pf_smem(sQ) + sw<HS>(r, c), qh + (int64_t)(ok ? r0 + r : 0) * vw.q_r + c * 8, ok);
+    const bool ok = r0 + r < T && (!EX || c * 8 < vw.dk);
+    pf_cp16(pf_smem(sQ) + sw<HS>(r, c), qh + (ok ? (int64_t)(r0 + r) * vw.q_r + c * 8 : 0), ok);
   }
   if constexpr (HK2 > 0) {
     for (int i = tid; i < kPfBM * CH2; i += kPfThreads) {
@@ -141,16 +147,34 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   // with a window the first rows of the tile decide where the key range starts (ragged positions grow with the row)
   const int tile_lo = window > 0 ? max(0, pos0 + r0 - window + 1) / kPfBN : 0;
   const int loA = window > 0 ? limA - window + 1 : 0, loB = window > 0 ? limB - window + 1 : 0;
+  // tiles in the order they are visited: those of the kept first positions that lie below the window's, then the window's
+  const int keep = EX ? vw.keep : 0;
+  const int kept_tiles = EX ? min((keep + kPfBN - 1) / kPfBN, tile_lo) : 0;
+  auto tile_at = [&](int it) { return it < kept_tiles ? it : tile_lo + it - kept_tiles; };
+  const int n_iter = kept_tiles + ntiles - tile_lo;
   const int warp_lo = window > 0 ? pos0 + r0 + warp * 16 - window + 1 : 0;     // lowest key any row of this warp sees
 
   auto load_kv = [&](int tile, int buf) {
     const int j0 = tile * kPfBN;
-    for (int i = tid; i < kPfBN * CH; i += kPfThreads) {
-      const int r = i / CH, c = i % CH;
-      const bool ok = j0 + r <= cta_lim;
-      const int64_t row = ok ? j0 + r : 0;
-      if constexpr (MODE != 2) pf_cp16(pf_smem(sK) + buf * KB + sw<HS>(r, c), kg + row * vw.k_r + c * 8, ok);
-      if constexpr (MODE != 1) pf_cp16(pf_smem(sV) + buf * KB + sw<HS>(r, c), vg + row * vw.v_r + c * 8, ok);
+    if constexpr (!EX) {
+      for (int i = tid; i < kPfBN * CH; i += kPfThreads) {
+        const int r = i / CH, c = i % CH;
+        const bool ok = j0 + r <= cta_lim;
+        const int64_t row = ok ? j0 + r : 0;
+        if constexpr (MODE != 2) pf_cp16(pf_smem(sK) + buf * KB + sw<HS>(r, c), kg + row * vw.k_r + c * 8, ok);
+        if constexpr (MODE != 1) pf_cp16(pf_smem(sV) + buf * KB + sw<HS>(r, c), vg + row * vw.v_r + c * 8, ok);
+      }
+    } else {
+      for (int i = tid; i < kPfBN * CH; i += kPfThreads) {
+        const int r = i / CH, c = i % CH;
+        const bool ok = j0 + r <= cta_lim && c * 8 < vw.dk;
+        pf_cp16(pf_smem(sK) + buf * KB + sw<HS>(r, c), kg + (ok ? (int64_t)(j0 + r) * vw.k_r + c * 8 : 0), ok);
+      }
+      for (int i = tid; i < kPfBN * CHV; i += kPfThreads) {
+        const int r = i / CHV, c = i % CHV;
+        const bool ok = j0 + r <= cta_lim && c * 8 < vw.dv;
+        pf_cp16(pf_smem(sV) + buf * VB + sw<HV>(r, c), vg + (ok ? (int64_t)(j0 + r) * vw.v_r + c * 8 : 0), ok);
+      }
     }
     if constexpr (HK2 > 0) {
       for (int i = tid; i < kPfBN * CH2; i += kPfThreads) {
@@ -161,11 +185,11 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     }
     pf_commit();
   };
-  load_kv(tile_lo, tile_lo & 1);
+  load_kv(tile_at(0), 0);
 
-  float o_acc[HS / 8][4];
+  float o_acc[HV / 8][4];
 #pragma unroll
-  for (int i = 0; i < HS / 8; ++i) o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f;
+  for (int i = 0; i < HV / 8; ++i) o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f;
   float mA = -INFINITY, mB = -INFINITY, lA = 0.f, lB = 0.f;
 
   // distance bias on the raw dot products: (s - r1 log2(1 + r2 dist) / scale_log2) * scale_log2 is the biased score in the log2 domain
@@ -193,16 +217,17 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   }
 
   const int warp_lim = wl;
-  for (int tile = tile_lo; tile < ntiles; ++tile) {
-    const int buf = tile & 1;
-    if (tile + 1 < ntiles) { load_kv(tile + 1, buf ^ 1); pf_wait<1>(); } else { pf_wait<0>(); }
+  const float sl = EX && vw.cap_in > 0.f ? 1.0f : scale_log2;   // capped scores are in the log2 domain already
+  for (int it = 0; it < n_iter; ++it) {
+    const int buf = it & 1, tile = tile_at(it);
+    if (it + 1 < n_iter) { load_kv(tile_at(it + 1), buf ^ 1); pf_wait<1>(); } else { pf_wait<0>(); }
     __syncthreads();
     const int j0 = tile * kPfBN;
-    if (j0 <= warp_lim && j0 + kPfBN > warp_lo) {   // warp-uniform: tiles entirely above this warp's rows, or below their windows, contribute nothing
+    if (j0 <= warp_lim && (j0 + kPfBN > warp_lo || (EX && j0 < keep))) {   // warp-uniform: tiles entirely above this warp's rows, or below their windows, contribute nothing
       float s[kPfBN / 8][4];
 #pragma unroll
       for (int i = 0; i < kPfBN / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-      const uint32_t kb = pf_smem(sK) + buf * KB, vb = pf_smem(sV) + buf * KB;
+      const uint32_t kb = pf_smem(sK) + buf * KB, vb = pf_smem(sV) + buf * VB;
       if constexpr (MODE == 2) {   // the scores were computed (and worked on) before: fetch this thread's share of the tile
         const float* tp = plane + (int64_t)tile * (kPfBM * kPfBN);
 #pragma unroll
@@ -241,6 +266,20 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
           }
         }
       }
+      if constexpr (EX) {
+        if (vw.cap_in > 0.f) {   // cap * tanh(x) = cap * (1 - 2 / (1 + e^2x)), here times log2(e); the reciprocal of infinity is 0
+#pragma unroll
+          for (int i = 0; i < kPfBN / 8; ++i) {
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+              float e, r;
+              asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(s[i][c] * vw.cap_in));
+              asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+              s[i][c] = fmaf(-2.0f * vw.cap_log2, r, vw.cap_log2);
+            }
+          }
+        }
+      }
       // causal limit + running maximum
       const bool need_mask = j0 + kPfBN - 1 > min(limA < 0 ? 0x7fffffff : limA, limB < 0 ? 0x7fffffff : limB) || limA < 0 || limB < 0 ||
                              (window > 0 && j0 < max(loA, loB));
@@ -271,10 +310,10 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
       for (int i = 0; i < kPfBN / 8; ++i) {
         if (need_mask) {
           const int j = j0 + i * 8 + 2 * tq;
-          if (j > limA || j < loA) s[i][0] = -INFINITY;
-          if (j + 1 > limA || j + 1 < loA) s[i][1] = -INFINITY;
-          if (j > limB || j < loB) s[i][2] = -INFINITY;
-          if (j + 1 > limB || j + 1 < loB) s[i][3] = -INFINITY;
+          if (j > limA || (j < loA && !(EX && j < keep))) s[i][0] = -INFINITY;
+          if (j + 1 > limA || (j + 1 < loA && !(EX && j + 1 < keep))) s[i][1] = -INFINITY;
+          if (j > limB || (j < loB && !(EX && j < keep))) s[i][2] = -INFINITY;
+          if (j + 1 > limB || (j + 1 < loB && !(EX && j + 1 < keep))) s[i][3] = -INFINITY;
         }
         tmA = fmaxf(tmA, fmaxf(s[i][0], s[i][1]));
         tmB = fmaxf(tmB, fmaxf(s[i][2], s[i][3]));
@@ -283,28 +322,28 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
       tmB = fmaxf(tmB, __shfl_xor_sync(0xffffffffu, tmB, 1)); tmB = fmaxf(tmB, __shfl_xor_sync(0xffffffffu, tmB, 2));
       const float nmA = fmaxf(mA, tmA), nmB = fmaxf(mB, tmB);
       // rows with nothing visible yet keep m = -inf: use 0 as the exponent origin so that exp2(-inf - 0) = 0
-      const float oA = nmA == -INFINITY ? 0.f : nmA * scale_log2, oB = nmB == -INFINITY ? 0.f : nmB * scale_log2;
-      const float cA = mA == -INFINITY ? 0.f : exp2f(mA * scale_log2 - oA), cB = mB == -INFINITY ? 0.f : exp2f(mB * scale_log2 - oB);
+      const float oA = nmA == -INFINITY ? 0.f : nmA * sl, oB = nmB == -INFINITY ? 0.f : nmB * sl;
+      const float cA = mA == -INFINITY ? 0.f : exp2f(mA * sl - oA), cB = mB == -INFINITY ? 0.f : exp2f(mB * sl - oB);
       mA = nmA; mB = nmB;
       float rsA = 0.f, rsB = 0.f;
       uint32_t pfr[kPfBN / 16][4];
 #pragma unroll
       for (int i = 0; i < kPfBN / 8; ++i) {
-        const float p0 = exp2f(fmaf(s[i][0], scale_log2, -oA)), p1 = exp2f(fmaf(s[i][1], scale_log2, -oA));
-        const float p2 = exp2f(fmaf(s[i][2], scale_log2, -oB)), p3 = exp2f(fmaf(s[i][3], scale_log2, -oB));
+        const float p0 = exp2f(fmaf(s[i][0], sl, -oA)), p1 = exp2f(fmaf(s[i][1], sl, -oA));
+        const float p2 = exp2f(fmaf(s[i][2], sl, -oB)), p3 = exp2f(fmaf(s[i][3], sl, -oB));
         rsA += p0 + p1; rsB += p2 + p3;
         pfr[i >> 1][(i & 1) * 2 + 0] = pack_bf16(p0, p1);
         pfr[i >> 1][(i & 1) * 2 + 1] = pack_bf16(p2, p3);
       }
       lA = lA * cA + rsA; lB = lB * cB + rsB;
 #pragma unroll
-      for (int i = 0; i < HS / 8; ++i) { o_acc[i][0] *= cA; o_acc[i][1] *= cA; o_acc[i][2] *= cB; o_acc[i][3] *= cB; }
+      for (int i = 0; i < HV / 8; ++i) { o_acc[i][0] *= cA; o_acc[i][1] *= cA; o_acc[i][2] *= cB; o_acc[i][3] *= cB; }
 #pragma unroll
       for (int ks = 0; ks < kPfBN / 16; ++ks) {
 #pragma unroll
-        for (int dp = 0; dp < HS / 16; ++dp) {
+        for (int dp = 0; dp < HV / 16; ++dp) {
           uint32_t vf[4];
-          ldsm_x4_t(vf, vb + sw<HS>(ks * 16 + (((lane >> 3) & 1) << 3) + (lane & 7), dp * 2 + (lane >> 4)));
+          ldsm_x4_t(vf, vb + sw<HV>(ks * 16 + (((lane >> 3) & 1) << 3) + (lane & 7), dp * 2 + (lane >> 4)));
           pf_mma(o_acc[2 * dp], pfr[ks], vf[0], vf[1]);
           pf_mma(o_acc[2 * dp + 1], pfr[ks], vf[2], vf[3]);
         }
@@ -320,12 +359,13 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   float iA = lA > 0.f ? 1.f / lA : 0.f, iB = lB > 0.f ? 1.f / lB : 0.f;
   if (vw.seqs && vw.sink) {   // the sink joins the denominator once: l is in units of exp2(m * scale_log2)
     const float sk = __bfloat162float(vw.sink[h]) * 1.4426950408889634f;
-    const float eA = mA == -INFINITY ? sk : fmaxf(mA * scale_log2, sk), eB = mB == -INFINITY ? sk : fmaxf(mB * scale_log2, sk);
-    const float cA = mA == -INFINITY ? 0.f : exp2f(mA * scale_log2 - eA), cB = mB == -INFINITY ? 0.f : exp2f(mB * scale_log2 - eB);
+    const float eA = mA == -INFINITY ? sk : fmaxf(mA * sl, sk), eB = mB == -INFINITY ? sk : fmaxf(mB * sl, sk);
+    const float cA = mA == -INFINITY ? 0.f : exp2f(mA * sl - eA), cB = mB == -INFINITY ? 0.f : exp2f(mB * sl - eB);
     iA = cA / (lA * cA + exp2f(sk - eA));
     iB = cB / (lB * cB + exp2f(sk - eB));
   }
   const int gmode = vw.seqs && vw.gate ? vw.gate_mode : 0;
+  const int dv = EX ? vw.dv : HV;
   // the gate's sigmoid with the fast exponential and reciprocal: the product is rounded to bf16 right after
   auto sigf = [](float z) -> float { return __fdividef(1.0f, 1.0f + __expf(-z)); };
   auto sigm = [&](const __nv_bfloat16* p) -> float { return sigf(__bfloat162float(*p)); };
@@ -342,30 +382,32 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     }
   };
   if (rowA < T) {
-    __nv_bfloat16* yr = y + (int64_t)b * vw.y_b + (qrow0 + rowA) * vw.y_r + (int64_t)h * HS;
+    __nv_bfloat16* yr = y + (int64_t)b * vw.y_b + (qrow0 + rowA) * vw.y_r + (int64_t)h * dv;
     const __nv_bfloat16* gr = gmode ? vw.gate + (qrow0 + rowA) * vw.gate_r : nullptr;
     if (gmode == 1) iA *= sigm(gr + h);
 #pragma unroll
-    for (int i = 0; i < HS / 8; ++i) {
+    for (int i = 0; i < HV / 8; ++i) {
+      if (EX && i * 8 >= dv) break;
       float a0 = o_acc[i][0] * iA, a1 = o_acc[i][1] * iA;
-      if (gmode == 2) gate2(gr + (int64_t)h * HS + i * 8 + 2 * tq, a0, a1);
+      if (gmode == 2) gate2(gr + (int64_t)h * dv + i * 8 + 2 * tq, a0, a1);
       *reinterpret_cast<uint32_t*>(yr + i * 8 + 2 * tq) = pack_bf16(a0, a1);
     }
   }
   if (rowB < T) {
-    __nv_bfloat16* yr = y + (int64_t)b * vw.y_b + (qrow0 + rowB) * vw.y_r + (int64_t)h * HS;
+    __nv_bfloat16* yr = y + (int64_t)b * vw.y_b + (qrow0 + rowB) * vw.y_r + (int64_t)h * dv;
     const __nv_bfloat16* gr = gmode ? vw.gate + (qrow0 + rowB) * vw.gate_r : nullptr;
     if (gmode == 1) iB *= sigm(gr + h);
 #pragma unroll
-    for (int i = 0; i < HS / 8; ++i) {
+    for (int i = 0; i < HV / 8; ++i) {
+      if (EX && i * 8 >= dv) break;
       float a0 = o_acc[i][2] * iB, a1 = o_acc[i][3] * iB;
-      if (gmode == 2) gate2(gr + (int64_t)h * HS + i * 8 + 2 * tq, a0, a1);
+      if (gmode == 2) gate2(gr + (int64_t)h * dv + i * 8 + 2 * tq, a0, a1);
       *reinterpret_cast<uint32_t*>(yr + i * 8 + 2 * tq) = pack_bf16(a0, a1);
     }
   }
 }
 
-template <int HS, typename PosT, int HK2 = 0, int MODE = 0>
+template <int HS, typename PosT, int HK2 = 0, int MODE = 0, int HV = HS, bool EX = false>
 cudaError_t launch_prefill(const void* q, const void* kc, const void* vc, const void* pos, void* y, int B, int T, int H, int G, int max_seq,
                            float scale, cudaStream_t st, const PfView* view = nullptr) {
   // default: q (B, H, T, HS), caches (B, G, max_seq, HS), y (B, T, H * HS)
@@ -373,17 +415,17 @@ cudaError_t launch_prefill(const void* q, const void* kc, const void* vc, const 
                          : PfView{(int64_t)H * T * HS, (int64_t)T * HS, HS, (int64_t)G * max_seq * HS, (int64_t)max_seq * HS, HS,
                                   (int64_t)G * max_seq * HS, (int64_t)max_seq * HS, HS, (int64_t)T * H * HS, (int64_t)H * HS, nullptr, 0, nullptr, 0,
                                   nullptr, 0, nullptr, 0, 0, nullptr, 0, 0, 0, 0};
-  const size_t tiles = (size_t)(kPfBM + 4 * kPfBN) * HS * 2 + (size_t)(kPfBM + 2 * kPfBN) * HK2 * 2;
+  const size_t tiles = (size_t)(kPfBM + 2 * kPfBN) * HS * 2 + (size_t)2 * kPfBN * HV * 2 + (size_t)(kPfBM + 2 * kPfBN) * HK2 * 2;
   const size_t smem = tiles + (size_t)vw.bias_n * sizeof(float);
   static PerDeviceOnce once;
   if (once.need()) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<HS, PosT, HK2, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_kernel<HS, PosT, HK2, MODE, HV, EX>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          (int)(tiles + kPfBiasTabMax * sizeof(float)));
     if (e != cudaSuccess) return e;
     once.done();
   }
   dim3 grid((T + kPfBM - 1) / kPfBM, H, B);
-  return launch(attn_prefill_kernel<HS, PosT, HK2, MODE>, grid, dim3(kPfThreads), smem, st, (const __nv_bfloat16*)q, (const __nv_bfloat16*)kc,
+  return launch(attn_prefill_kernel<HS, PosT, HK2, MODE, HV, EX>, grid, dim3(kPfThreads), smem, st, (const __nv_bfloat16*)q, (const __nv_bfloat16*)kc,
                 (const __nv_bfloat16*)vc, (const PosT*)pos, (__nv_bfloat16*)y, T, H, G, max_seq, scale * 1.4426950408889634f, vw);
 }
 
@@ -542,6 +584,35 @@ extern "C" int b200_attn_prefill_window_ex(const void* q, int64_t ldq, const voi
   cudaStream_t st = (cudaStream_t)stream;
   if (head_size == 128) B200_CUDA((launch_prefill<128, int32_t>(q, k, v, nullptr, y, n_seqs, max_q_len, n_head, n_kv_head, 0, scale, st, &vw)));
   else B200_CUDA((launch_prefill<64, int32_t>(q, k, v, nullptr, y, n_seqs, max_q_len, n_head, n_kv_head, 0, scale, st, &vw)));
+  return B200_OK;
+}
+
+// The same tiles with kept first positions, a soft cap, and query / key and value sizes of their own (multiples of 8 up to 128, padded
+// with zeros to 64 or 128 in shared memory), described as b200_window_attn describes them; the sequences start in this step.
+extern "C" int b200_window_attn_tiles(const b200_window_attn_args* a, b200_stream_t stream) {
+  B200_CHECK_ARG(a && a->q && a->k && a->v && a->out && a->seqs, "b200_window_attn_tiles: null pointer");
+  B200_CHECK_ARG(!a->dist_r1 && !a->dist_r2, "b200_window_attn_tiles: no distance bias here");
+  B200_CHECK_ARG(a->gate_mode >= 0 && a->gate_mode <= 2 && (a->gate_mode == 0 || a->gate), "b200_window_attn_tiles: bad gate");
+  B200_CHECK_ARG(a->n_seqs > 0 && a->n_seqs <= 65535 && a->max_q_len > 0 && a->n_head > 0 && a->n_head <= 65535 && a->n_kv_head > 0 &&
+                     a->n_head % a->n_kv_head == 0 && a->window > 0 && a->keep >= 0 && a->softcap >= 0.f && a->scale > 0.f,
+                 "b200_window_attn_tiles: bad shape");
+  B200_CHECK_ARG(a->dtype == B200_BF16 && a->dk > 0 && a->dk <= 128 && a->dk % 8 == 0 && a->dv > 0 && a->dv <= 128 && a->dv % 8 == 0,
+                 "b200_window_attn_tiles: bf16 heads of multiples of 8 numbers, at most 128");
+  B200_CHECK_ARG(((a->ldq | a->ldk | a->ldv) & 7) == 0 && (a->ldo & 1) == 0, "b200_window_attn_tiles: leading dimensions must be multiples of 8 elements");
+  B200_CHECK_ARG(((reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->k) | reinterpret_cast<uintptr_t>(a->v) |
+                   reinterpret_cast<uintptr_t>(a->seqs)) & 15) == 0 && (reinterpret_cast<uintptr_t>(a->out) & 3) == 0,
+                 "b200_window_attn_tiles: operands must be 16-byte aligned");
+  constexpr float kLog2e = 1.4426950408889634f;
+  const PfView vw{0, a->dk, a->ldq, 0, a->dk, a->ldk, 0, a->dv, a->ldv, 0, a->ldo, reinterpret_cast<const int4*>(a->seqs), a->window,
+                  reinterpret_cast<const __nv_bfloat16*>(a->sink), 1, nullptr, 0, a->gate_mode ? reinterpret_cast<const __nv_bfloat16*>(a->gate) : nullptr,
+                  a->ldg, a->gate_mode, nullptr, 0, 0, 0, 0, nullptr, nullptr, 0, a->dk, a->dv, a->keep, a->softcap * kLog2e,
+                  a->softcap > 0.f ? 2.0f * a->scale / a->softcap * kLog2e : 0.f};
+  cudaStream_t st = (cudaStream_t)stream;
+  const int H = a->n_head, G = a->n_kv_head;
+  if (a->dk > 64 && a->dv > 64) B200_CUDA((launch_prefill<128, int32_t, 0, 0, 128, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+  else if (a->dk > 64) B200_CUDA((launch_prefill<128, int32_t, 0, 0, 64, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+  else if (a->dv > 64) B200_CUDA((launch_prefill<64, int32_t, 0, 0, 128, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+  else B200_CUDA((launch_prefill<64, int32_t, 0, 0, 64, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
   return B200_OK;
 }
 

@@ -49,8 +49,8 @@ __global__ void __launch_bounds__(kRowThreads) embed_pos_kernel(const int* __res
   }
 }
 
-// out[orow] = in[irow] / sqrt(mean(in[irow]^2) + eps) * (weight or 1 + weight); blockIdx.y picks one of two segments so
-// that the two norms that follow one fused down-projection run as a single launch
+// out[orow] = in[irow] / sqrt(mean(in[irow]^2) + eps) * (weight or 1 + weight), with `center` of the row minus its mean (a layer norm
+// without bias); blockIdx.y picks one of two segments so that the two norms that follow one fused down-projection run as a single launch
 struct RmsSeg {
   const void* in;
   const void* weight;
@@ -58,7 +58,7 @@ struct RmsSeg {
   const int64_t* in_rows;   // NULL: row index itself
   const int64_t* out_rows;  // NULL: row index itself
   int64_t ld_in, ld_out;
-  int d, plus_one;
+  int d, plus_one, center;
 };
 
 template <typename TI, typename TO>
@@ -75,17 +75,32 @@ __global__ void __launch_bounds__(kRowThreads) rms_rows_kernel(RmsSeg s0, RmsSeg
   TO* yr = reinterpret_cast<TO*>(s.out) + orow * s.ld_out;
   const bool vec = vec8_ok(s.d, xr, w, yr);
   const float one = s.plus_one ? 1.0f : 0.0f;
+  float mu = 0.f;
+  if (s.center) {
+    float sum = 0.f;
+    if (vec) {
+      for (int i = threadIdx.x * 8; i < s.d; i += kRowThreads * 8) {
+        float v[8];
+        load8(xr + i, v);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sum += v[j];
+      }
+    } else {
+      for (int i = threadIdx.x; i < s.d; i += kRowThreads) sum += load_as_float(xr, i);
+    }
+    mu = cta_sum(sum, s_part) / (float)s.d;
+  }
   float ss = 0.f;
   if (vec) {
     for (int i = threadIdx.x * 8; i < s.d; i += kRowThreads * 8) {
       float v[8];
       load8(xr + i, v);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
+      for (int j = 0; j < 8; ++j) ss = fmaf(v[j] - mu, v[j] - mu, ss);
     }
   } else {
     for (int i = threadIdx.x; i < s.d; i += kRowThreads) {
-      const float v = load_as_float(xr, i);
+      const float v = load_as_float(xr, i) - mu;
       ss = fmaf(v, v, ss);
     }
   }
@@ -96,11 +111,11 @@ __global__ void __launch_bounds__(kRowThreads) rms_rows_kernel(RmsSeg s0, RmsSeg
       load8(xr + i, v);
       load8(w + i, g);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) v[j] = v[j] * rstd * (g[j] + one);
+      for (int j = 0; j < 8; ++j) v[j] = (v[j] - mu) * rstd * (g[j] + one);
       store8(yr + i, v);
     }
   } else {
-    for (int i = threadIdx.x; i < s.d; i += kRowThreads) store_from_float(yr, i, load_as_float(xr, i) * rstd * (load_as_float(w, i) + one));
+    for (int i = threadIdx.x; i < s.d; i += kRowThreads) store_from_float(yr, i, (load_as_float(xr, i) - mu) * rstd * (load_as_float(w, i) + one));
   }
 }
 
@@ -156,7 +171,8 @@ __global__ void __launch_bounds__(kRowThreads) residual_norm_add_kernel(const T*
 //   y    = y0                                   (one branch)
 //        | (norm(y0) * w0 + norm(y1) * w1) / 2  (two mixers side by side, each RMS-normed over the width with its own weight)
 //   x   += norm(y) * post_w  [+ extra]          (fp32 stream; `extra`: e.g. the embedding re-entering before a repeated pass)
-//   act  = T(norm(x) * pre_w)                   (input of the next sublayer; skipped without pre_w)
+//   cast = T(x)                                 (optional copy in the matrix-product dtype)
+//   act  = T(norm(x) * pre_w)                   (input of the next sublayer; skipped without pre_w; with pre_center norm(x - mean(x)))
 // norm(z) = z / sqrt(mean(z^2) + eps), statistics in fp32.  One CTA per row; the row lives in shared memory between the passes.
 struct SandwichArgs {
   const void* y0; const void* w0; const void* y1; const void* w1;
@@ -164,6 +180,8 @@ struct SandwichArgs {
   float* x; void* act;
   int d;
   float eps;
+  int pre_center;
+  void* cast;
 };
 
 template <typename T>
@@ -183,8 +201,9 @@ __global__ void __launch_bounds__(kRowThreads) sandwich_residual_kernel(Sandwich
   float* xr = A.x + row * d;
   const float* ex = A.extra ? A.extra + row * d : nullptr;
   T* ar = nw ? reinterpret_cast<T*>(A.act) + row * d : nullptr;
+  T* cr = A.cast ? reinterpret_cast<T*>(A.cast) + row * d : nullptr;
   // eight elements per access when every row and weight starts on a 16-byte boundary (d a multiple of 8, aligned bases)
-  const bool vec = vec8_ok(d, A.y0, A.y1, A.w0, A.w1) && vec8_ok(d, A.post_w, A.pre_w, A.x, A.act) && vec8_ok(d, A.extra);
+  const bool vec = vec8_ok(d, A.y0, A.y1, A.w0, A.w1) && vec8_ok(d, A.post_w, A.pre_w, A.x, A.act) && vec8_ok(d, A.extra, A.cast);
   float s0 = 0.f, s1 = 0.f;
   if (vec) {
     for (int i = threadIdx.x * 8; i < d; i += kRowThreads * 8) {
@@ -243,7 +262,8 @@ __global__ void __launch_bounds__(kRowThreads) sandwich_residual_kernel(Sandwich
   }
   float rp = 1.0f;
   if (pw) rp = 1.0f / sqrtf(cta_sum(ss, s_part) / (float)d + A.eps);
-  float sx = 0.f;
+  const bool center = A.pre_center != 0;
+  float sx = 0.f;   // sum of squares, or of the numbers themselves when the mean is to come off first
   // each thread touches only the elements it wrote: no barrier needed between the passes over sw_row
   if (vec) {
     for (int i = threadIdx.x * 8; i < d; i += kRowThreads * 8) {
@@ -257,31 +277,46 @@ __global__ void __launch_bounds__(kRowThreads) sandwich_residual_kernel(Sandwich
         if (ex) v += e[j];
         xv[j] = v;
         sw_row[i + j] = v;
-        sx = fmaf(v, v, sx);
+        sx = center ? sx + v : fmaf(v, v, sx);
       }
       store8(xr + i, xv);
+      if (cr) store8(cr + i, xv);
     }
   } else {
     for (int i = threadIdx.x; i < d; i += kRowThreads) {
       float v = xr[i] + (pw ? sw_row[i] * rp * load_as_float(pw, i) : sw_row[i]);
       if (ex) v += ex[i];
       xr[i] = v;
+      if (cr) store_from_float(cr, i, v);
       sw_row[i] = v;
-      sx = fmaf(v, v, sx);
+      sx = center ? sx + v : fmaf(v, v, sx);
     }
   }
   if (!nw) return;
+  float mu = 0.f;
+  if (center) {
+    mu = cta_sum(sx, s_part) / (float)d;
+    sx = 0.f;
+    if (vec) {
+      for (int i = threadIdx.x * 8; i < d; i += kRowThreads * 8) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sx = fmaf(sw_row[i + j] - mu, sw_row[i + j] - mu, sx);
+      }
+    } else {
+      for (int i = threadIdx.x; i < d; i += kRowThreads) sx = fmaf(sw_row[i] - mu, sw_row[i] - mu, sx);
+    }
+  }
   const float rn = 1.0f / sqrtf(cta_sum(sx, s_part) / (float)d + A.eps);
   if (vec) {
     for (int i = threadIdx.x * 8; i < d; i += kRowThreads * 8) {
       float g[8], o[8];
       load8(nw + i, g);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) o[j] = sw_row[i + j] * rn * g[j];
+      for (int j = 0; j < 8; ++j) o[j] = (sw_row[i + j] - mu) * rn * g[j];
       store8(ar + i, o);
     }
   } else {
-    for (int i = threadIdx.x; i < d; i += kRowThreads) store_from_float(ar, i, sw_row[i] * rn * load_as_float(nw, i));
+    for (int i = threadIdx.x; i < d; i += kRowThreads) store_from_float(ar, i, (sw_row[i] - mu) * rn * load_as_float(nw, i));
   }
 }
 
@@ -310,6 +345,22 @@ __global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ in, T* _
   for (int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x; i < n; i += (int64_t)gridDim.x * 256) {
     const int64_t r = i / ff, c = i - r * ff;
     store_from_float(out, i, activate(load_as_float(in, r * 2 * ff + c), kind) * load_as_float(in, r * 2 * ff + ff + c));
+  }
+}
+
+// out[r, c] = act(z[r, c]) * table[token[r], off + c]: a row's projection, activated, times its token's entry of a second embedding
+// table (`cols` neighbouring columns from `off` on)
+template <typename T>
+__global__ void __launch_bounds__(256) token_gate_kernel(const T* __restrict__ z, int64_t ldz, const int* __restrict__ tokens, const T* __restrict__ table,
+                                                         int64_t ld_table, int64_t off, int vocab, T* __restrict__ out, int64_t rows, int cols, int kind) {
+  griddep_launch();
+  griddep_wait();
+  const int64_t n = rows * cols;
+  for (int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x; i < n; i += (int64_t)gridDim.x * 256) {
+    const int64_t r = i / cols, c = i - r * cols;
+    int tok = tokens[r];
+    tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);  // never read out of bounds
+    store_from_float(out, i, activate(load_as_float(z, r * ldz + c), kind) * load_as_float(table, tok * ld_table + off + c));
   }
 }
 
@@ -532,7 +583,7 @@ int b200_rms_rows(const b200_rms_rows_seg* segs, int n_segs, int64_t rows, float
   for (int i = 0; i < 2; ++i) {
     const b200_rms_rows_seg& a = segs[i < n_segs ? i : 0];
     B200_CHECK_ARG(a.in && a.weight && a.out && a.d > 0, "b200_rms_rows: null pointer or empty row");
-    s[i] = RmsSeg{a.in, a.weight, a.out, a.in_rows, a.out_rows, a.ld_in, a.ld_out, a.d, a.plus_one};
+    s[i] = RmsSeg{a.in, a.weight, a.out, a.in_rows, a.out_rows, a.ld_in, a.ld_out, a.d, a.plus_one, a.center};
   }
   const dim3 grid((unsigned)rows, (unsigned)n_segs), block(kRowThreads);
   cudaStream_t st = (cudaStream_t)stream;
@@ -586,7 +637,7 @@ int b200_sandwich_residual(const b200_sandwich_args* a, b200_stream_t stream) {
   B200_CHECK_ARG(!a->y1 || (a->w0 && a->w1), "b200_sandwich_residual: two branches need their two norm weights");
   B200_CHECK_ARG(!a->pre_w || a->act, "b200_sandwich_residual: the next sublayer's norm needs somewhere to go");
   B200_CHECK_ARG(a->rows > 0 && a->rows <= 0x7fffffff && a->d > 0 && (size_t)a->d * sizeof(float) <= 160 * 1024, "b200_sandwich_residual: bad shape");
-  const SandwichArgs A{a->y0, a->w0, a->y1, a->w1, a->post_w, a->extra, a->pre_w, a->x, a->act, a->d, a->eps};
+  const SandwichArgs A{a->y0, a->w0, a->y1, a->w1, a->post_w, a->extra, a->pre_w, a->x, a->act, a->d, a->eps, a->pre_center, a->cast};
   const size_t smem = (size_t)a->d * sizeof(float);
   B200_FLOAT_TYPES(a->dtype, T, {
     static PerDeviceOnce once;
@@ -614,6 +665,18 @@ int b200_glu(const void* in, void* out, int64_t rows, int ff, int kind, int dtyp
   const int64_t cap = (int64_t)sm_count() * 16;
   if (blocks > cap) blocks = cap;
   B200_FLOAT_TYPES(dtype, T, B200_CUDA(launch(glu_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, (const T*)in, (T*)out, rows, ff, kind)));
+  return B200_OK;
+}
+
+int b200_token_gate(const void* z, int64_t ldz, const int32_t* tokens, const void* table, int64_t ld_table, int64_t off, int vocab, void* out,
+                    int64_t rows, int cols, int kind, int dtype, b200_stream_t stream) {
+  B200_CHECK_ARG(z && tokens && table && out && rows > 0 && cols > 0 && vocab > 0 && kind >= 0 && kind <= 3, "b200_token_gate: bad argument");
+  B200_CHECK_ARG(off >= 0 && off + cols <= ld_table && ldz >= cols, "b200_token_gate: the columns do not fit the table's rows");
+  int64_t blocks = (rows * cols + 255) / 256;
+  const int64_t cap = (int64_t)sm_count() * 16;
+  if (blocks > cap) blocks = cap;
+  B200_FLOAT_TYPES(dtype, T, B200_CUDA(launch(token_gate_kernel<T>, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, (const T*)z, ldz, tokens,
+                                               (const T*)table, ld_table, off, vocab, (T*)out, rows, cols, kind)));
   return B200_OK;
 }
 

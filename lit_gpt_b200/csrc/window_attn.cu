@@ -2,13 +2,14 @@
 //
 //   row at position i sees positions j with 0 <= i - j < window;  p_j = exp(s_j) / (exp(sink_h) + sum_j' exp(s_j')),
 //   s_j = (q . k_j) * scale.  The sink is one learned logit per head with no key and no value: it only takes probability.
-//   Optional: a distance bias, s_j -= r1_h * ln(1 + r2_h * (i - j)) with two numbers per head, and a sigmoid output gate read from
+//   Optional: kept first tokens (positions j < keep stay visible forever), a soft cap, s_j <- cap * tanh(s_j / cap), a distance bias, s_j -= r1_h * ln(1 + r2_h * (i - j)) with two numbers per head, and a sigmoid output gate read from
 //   raw projections of the row (one per head, or one per output number).
 //
 // Grouped heads (query head h reads key-value head h / (H / G)), separate query-key (dk) and value (dv) sizes, any sizes,
 // operands bf16 or fp32, all arithmetic fp32 with a running maximum.
 //
-// Only the last `ring` >= window positions of a sequence are kept: position p lives in row p % ring of the sequence's slot.
+// Only the first `keep` and the last `ring` >= window positions of a sequence are held: position p lives in row p of the sequence's
+// slot (p < keep), else in row keep + (p - keep) % ring.
 // A step's own keys and values are read from the step's packed rows (k, v), older ones from the ring, so one kernel serves
 // a whole prompt, a later portion of one and single decoded tokens; the step's last rows enter the ring AFTERWARDS (a long
 // step would otherwise overwrite ring rows that its first queries still need): b200_ring_store after the tiled kernel, the
@@ -45,7 +46,15 @@ struct WaArgs {
   const void* gate;                 // raw gate projections, rows ldg apart (NULL: none)
   int64_t ldg;
   int gate_mode;                    // 1: column h of the gate row; 2: column h * dv + c
+  int keep;                         // first positions that never leave the window, nor the cache
+  float cap_log2, inv_cap;          // soft cap: cap * log2(e), and 1 / (cap * log2(e)); inv_cap 0: none
 };
+
+// cache row of position p, within the rows of all slots
+__device__ __forceinline__ int64_t wa_ring_row(int slot, int ring, int keep, int p) {
+  return (int64_t)slot * (ring + keep) + (p < keep ? p : keep + (p - keep) % ring);
+}
+__device__ __forceinline__ float wa_cap(const WaArgs& A, float s) { return A.inv_cap > 0.f ? A.cap_log2 * tanhf(s * A.inv_cap) : s; }
 
 // output gate of one number: sigmoid of the raw projection
 template <typename T>
@@ -106,24 +115,27 @@ __global__ void __launch_bounds__(kWaThreads) window_attn_kernel(WaArgs A) {
   const float r1h = biased ? load_as_float(reinterpret_cast<const T*>(A.r1), h) : 0.f;
   const float r2h = biased ? load_as_float(reinterpret_cast<const T*>(A.r2), h) : 0.f;
 
-  for (int j0 = key_lo; j0 < key_hi; j0 += kWaBN) {
+  // key tiles: the kept first positions below the window, then the window
+  const int keep_hi = min(A.keep, key_lo);
+  for (int j0 = keep_hi > 0 ? 0 : key_lo; j0 < key_hi; j0 = (j0 < keep_hi && j0 + kWaBN >= keep_hi) ? key_lo : j0 + kWaBN) {
+    const int j1 = j0 < keep_hi ? keep_hi : key_hi;              // one past the last key of this run
     __syncthreads();
     for (int idx = tid; idx < kWaBN * dkp; idx += kWaThreads) {
       const int j = idx / dkp, d = idx - j * dkp;
       const int p = j0 + j;
       float val = 0.f;
-      if (p < key_hi && d < dk)
+      if (p < j1 && d < dk)
         val = p >= pos0 ? load_as_float(k, (int64_t)(first + p - pos0) * A.ldk + (int64_t)g * dk + d)
-                        : load_as_float(kr, ((int64_t)slot * A.ring + p % A.ring) * G * dk + (int64_t)g * dk + d);
+                        : load_as_float(kr, wa_ring_row(slot, A.ring, A.keep, p) * G * dk + (int64_t)g * dk + d);
       Ks[idx] = val;
     }
     for (int idx = tid; idx < kWaBN * kWaDV; idx += kWaThreads) {
       const int j = idx / kWaDV, c = idx - j * kWaDV;
       const int p = j0 + j;
       float val = 0.f;
-      if (p < key_hi && c < dvc)
+      if (p < j1 && c < dvc)
         val = p >= pos0 ? load_as_float(v, (int64_t)(first + p - pos0) * A.ldv + (int64_t)g * dv + c0 + c)
-                        : load_as_float(vr, ((int64_t)slot * A.ring + p % A.ring) * G * dv + (int64_t)g * dv + c0 + c);
+                        : load_as_float(vr, wa_ring_row(slot, A.ring, A.keep, p) * G * dv + (int64_t)g * dv + c0 + c);
       Vs[idx] = val;
     }
     __syncthreads();
@@ -156,7 +168,9 @@ __global__ void __launch_bounds__(kWaThreads) window_attn_kernel(WaArgs A) {
 #pragma unroll
       for (int b = 0; b < 4; ++b) {
         const int p = j0 + tx + 16 * b;
-        if (p > lim[a] || p <= lim[a] - A.window) s[a][b] = -INFINITY;   // ahead of the row, or fallen out of its window
+        s[a][b] = wa_cap(A, s[a][b]);
+        // ahead of the row (or of this run of keys), or fallen out of the row's window and not kept
+        if (p > lim[a] || p >= j1 || (p <= lim[a] - A.window && p >= A.keep)) s[a][b] = -INFINITY;
         else if (biased) s[a][b] -= r1h * log2f(fmaf(r2h, (float)(lim[a] - p), 1.0f));
         mx = fmaxf(mx, s[a][b]);
       }
@@ -235,21 +249,23 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
   const int4 sq = A.seqs[blockIdx.y];
   const int row = sq.x, pos = sq.z, slot = sq.w;
   const int dk = A.dk, dv = A.dv;
-  const int lo = max(0, pos - A.window + 1), n = pos - lo + 1;     // visible positions lo .. pos
+  const int lo = max(0, pos - A.window + 1);
+  const int nk = min(A.keep, lo), n = nk + pos - lo + 1;           // visible: 0 .. nk - 1 (kept), then lo .. pos; entry j of n:
+  auto position = [&](int j) { return j < nk ? j : lo + j - nk; };
   float* const qs = wd_smem;                        // [dk rounded up to 8]
-  float* const sc = qs + ((dk + 7) & ~7);           // [window rounded up to 4]
-  float* const part = sc + ((A.window + 3) & ~3);   // [value rows][dv]
+  float* const sc = qs + ((dk + 7) & ~7);           // [window + keep rounded up to 4]
+  float* const part = sc + ((A.window + A.keep + 3) & ~3);   // [value rows][dv]
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const T* const kr = reinterpret_cast<const T*>(A.k_ring);
   const T* const vr = reinterpret_cast<const T*>(A.v_ring);
   const T* const k_now = reinterpret_cast<const T*>(A.k) + (int64_t)row * A.ldk + (int64_t)g * dk;
   const T* const v_now = reinterpret_cast<const T*>(A.v) + (int64_t)row * A.ldv + (int64_t)g * dv;
-  auto key_row = [&](int p) { return p == pos ? k_now : kr + ((int64_t)slot * A.ring + p % A.ring) * G * dk + (int64_t)g * dk; };
-  auto value_row = [&](int p) { return p == pos ? v_now : vr + ((int64_t)slot * A.ring + p % A.ring) * G * dv + (int64_t)g * dv; };
+  auto key_row = [&](int p) { return p == pos ? k_now : kr + wa_ring_row(slot, A.ring, A.keep, p) * G * dk + (int64_t)g * dk; };
+  auto value_row = [&](int p) { return p == pos ? v_now : vr + wa_ring_row(slot, A.ring, A.keep, p) * G * dv + (int64_t)g * dv; };
   for (int d = tid; d < dk; d += kWdThreads) qs[d] = load_as_float(reinterpret_cast<const T*>(A.q), (int64_t)row * A.ldq + (int64_t)h * dk + d) * A.scale_log2;
   __syncthreads();
   float mx = -INFINITY;
-  // distance bias in the log2 domain; visible position j of n lies n - 1 - j behind the row
+  // distance bias in the log2 domain
   const bool biased = A.r1 != nullptr;
   const float r1h = biased ? load_as_float(reinterpret_cast<const T*>(A.r1), h) : 0.f;
   const float r2h = biased ? load_as_float(reinterpret_cast<const T*>(A.r2), h) : 0.f;
@@ -263,7 +279,7 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
 #pragma unroll
         for (int u = 0; u < U; ++u) {
           const int j = jb + u * KG + grp;
-          const T* kp = key_row(lo + min(j, n - 1));
+          const T* kp = key_row(position(min(j, n - 1)));
 #pragma unroll
           for (int pc = 0; pc < 2; ++pc) {
             const int c = sub * 8 + pc * 64;
@@ -292,7 +308,7 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
           const int j = jb + u * KG + grp;
           acc[u] = 0.f;
           if (j < n) {
-            const T* kp = key_row(lo + j);
+            const T* kp = key_row(position(j));
             for (int c = sub * 8; c < dk; c += 64) {
               float f[8];
               load8(kp + c, f);
@@ -310,7 +326,8 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
         a += __shfl_xor_sync(0xffffffffu, a, 2);
         a += __shfl_xor_sync(0xffffffffu, a, 1);
         if (j < n) {
-          if (biased) a -= r1h * log2f(fmaf(r2h, (float)(n - 1 - j), 1.0f));
+          a = wa_cap(A, a);
+          if (biased) a -= r1h * log2f(fmaf(r2h, (float)(pos - position(j)), 1.0f));
           if (sub == 0) sc[j] = a;
           mx = fmaxf(mx, a);
         }
@@ -318,11 +335,11 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
     }
   } else {
     for (int j = warp; j < n; j += kWdWarps) {       // one warp per key
-      const T* kp = key_row(lo + j);
+      const T* kp = key_row(position(j));
       float acc = 0.f;
       for (int d = lane; d < dk; d += 32) acc = fmaf(qs[d], load_as_float(kp, d), acc);
-      acc = warp_sum(acc);
-      if (biased) acc -= r1h * log2f(fmaf(r2h, (float)(n - 1 - j), 1.0f));
+      acc = wa_cap(A, warp_sum(acc));
+      if (biased) acc -= r1h * log2f(fmaf(r2h, (float)(pos - position(j)), 1.0f));
       if (lane == 0) sc[j] = acc;
       mx = fmaxf(mx, acc);
     }
@@ -357,7 +374,7 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
 #pragma unroll 4
       for (int j = rj; j < n; j += vrows) {
         float f[8];
-        load8(value_row(lo + j) + cg * 8, f);
+        load8(value_row(position(j)) + cg * 8, f);
         const float p = sc[j];
 #pragma unroll
         for (int e = 0; e < 8; ++e) acc[e] = fmaf(p, f[e], acc[e]);
@@ -368,7 +385,7 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
   } else {
     for (int c = lane; c < dv; c += 32) {
       float acc = 0.f;
-      for (int j = warp; j < n; j += kWdWarps) acc = fmaf(sc[j], load_as_float(value_row(lo + j), c), acc);
+      for (int j = warp; j < n; j += kWdWarps) acc = fmaf(sc[j], load_as_float(value_row(position(j)), c), acc);
       part[warp * dv + c] = acc;
     }
   }
@@ -378,28 +395,28 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
     for (int r = 0; r < vrows; ++r) t += part[r * dv + c];
     store_from_float(reinterpret_cast<T*>(A.out), (int64_t)row * A.ldo + (int64_t)h * dv + c, t * inv * wa_gate<T>(A, row, h, c));
   }
-  // The row's own key and value enter the ring here: they replace position pos - ring, which no row of this step can see
+  // The row's own key and value enter the ring here: they replace position pos - ring (kept rows are never replaced), which no row of this step can see
   // (ring >= window), and every CTA reads the current position from the step's rows, never from the ring.
   if (A.store_ring && h % (A.n_head / G) == 0) {
-    T* kd = const_cast<T*>(kr) + ((int64_t)slot * A.ring + pos % A.ring) * G * dk + (int64_t)g * dk;
-    T* vd = const_cast<T*>(vr) + ((int64_t)slot * A.ring + pos % A.ring) * G * dv + (int64_t)g * dv;
+    T* kd = const_cast<T*>(kr) + wa_ring_row(slot, A.ring, A.keep, pos) * G * dk + (int64_t)g * dk;
+    T* vd = const_cast<T*>(vr) + wa_ring_row(slot, A.ring, A.keep, pos) * G * dv + (int64_t)g * dv;
     for (int d = tid; d < dk; d += kWdThreads) kd[d] = k_now[d];
     for (int c = tid; c < dv; c += kWdThreads) vd[c] = v_now[c];
   }
 }
 
-// ring[slot][p % ring] <- row, for the rows whose position p is among the sequence's last `ring`
+// ring[slot][row of p] <- row, for the rows whose position p is among the sequence's first `keep` or last `ring`
 template <typename T>
 __global__ void __launch_bounds__(128) ring_store_kernel(const T* __restrict__ k, int64_t ldk, const T* __restrict__ v, int64_t ldv,
-                                                         T* __restrict__ k_ring, T* __restrict__ v_ring, int ring, int kcols, int vcols,
+                                                         T* __restrict__ k_ring, T* __restrict__ v_ring, int ring, int keep, int kcols, int vcols,
                                                          const int4* __restrict__ seqs, const int* __restrict__ row_seq) {
   griddep_launch();
   griddep_wait();
   const int64_t row = blockIdx.x;
   const int4 sq = seqs[row_seq[row]];
   const int p = sq.z + (int)(row - sq.x), end = sq.z + sq.y;
-  if (p < end - ring) return;
-  const int64_t dst = (int64_t)sq.w * ring + p % ring;
+  if (p >= keep && p < end - ring) return;
+  const int64_t dst = wa_ring_row(sq.w, ring, keep, p);
   for (int i = threadIdx.x; i < kcols; i += 128) k_ring[dst * kcols + i] = k[row * ldk + i];
   for (int i = threadIdx.x; i < vcols; i += 128) v_ring[dst * vcols + i] = v[row * ldv + i];
 }
@@ -427,17 +444,19 @@ int b200_window_attn(const b200_window_attn_args* a, b200_stream_t stream) {
                  "b200_window_attn: bad head shape (query-key size up to 512)");
   B200_CHECK_ARG(a->window > 0 && a->ring >= a->window && a->k_ring && a->v_ring, "b200_window_attn: the ring must hold at least one window");
   B200_CHECK_ARG((reinterpret_cast<uintptr_t>(a->seqs) & 15) == 0, "b200_window_attn: seqs must be 16-byte aligned");
+  B200_CHECK_ARG(a->keep >= 0 && a->keep <= (1 << 20) && a->softcap >= 0.f, "b200_window_attn: bad kept tokens or soft cap");
   B200_CHECK_ARG(!a->dist_r1 == !a->dist_r2, "b200_window_attn: the distance bias needs both of its numbers per head");
   B200_CHECK_ARG(a->gate_mode >= 0 && a->gate_mode <= 2 && (a->gate_mode == 0 || a->gate), "b200_window_attn: bad gate");
   const WaArgs A{a->q, a->k, a->v, a->out, a->ldq, a->ldk, a->ldv, a->ldo, a->k_ring, a->v_ring, a->sink, reinterpret_cast<const int4*>(a->seqs),
                  a->ring, a->n_head, a->n_kv_head, a->dk, a->dv, a->window, a->scale * kLog2e, a->row_seq != nullptr,
-                 a->dist_r1, a->dist_r2, a->gate_mode ? a->gate : nullptr, a->ldg, a->gate_mode};
+                 a->dist_r1, a->dist_r2, a->gate_mode ? a->gate : nullptr, a->ldg, a->gate_mode, a->keep, a->softcap * kLog2e,
+                 a->softcap > 0.f ? 1.0f / (a->softcap * kLog2e) : 0.f};
   cudaStream_t st = (cudaStream_t)stream;
   const size_t esz = a->dtype == B200_F32 ? 4 : 2;
   auto aligned = [&](const void* p, int64_t ld) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0 && (ld * esz) % 16 == 0; };
   const bool vec = a->dk % 8 == 0 && a->dv % 8 == 0 && a->dv <= 8 * kWdThreads && aligned(a->k, a->ldk) && aligned(a->v, a->ldv) &&
                    aligned(a->k_ring, 8) && aligned(a->v_ring, 8);
-  const size_t smem_d = (size_t)(((a->dk + 7) & ~7) + ((a->window + 3) & ~3) + wd_value_rows(a->dv, vec) * a->dv) * sizeof(float);
+  const size_t smem_d = (size_t)(((a->dk + 7) & ~7) + ((a->window + a->keep + 3) & ~3) + wd_value_rows(a->dv, vec) * a->dv) * sizeof(float);
   if (a->max_q_len == 1 && !g_wa_force_tiled && smem_d <= 160 * 1024 && a->n_head <= 65535) {
     B200_FLOAT_TYPES(a->dtype, T, {
       static PerDeviceOnce once;
@@ -465,18 +484,23 @@ int b200_window_attn(const b200_window_attn_args* a, b200_stream_t stream) {
     B200_CUDA(launch(window_attn_kernel<T>, grid, dim3(kWaThreads), smem, st, A));
   });
   if (a->row_seq)
-    return b200_ring_store(a->k, a->ldk, a->v, a->ldv, const_cast<void*>(a->k_ring), const_cast<void*>(a->v_ring), a->ring, a->n_kv_head * a->dk,
-                           a->n_kv_head * a->dv, a->seqs, a->row_seq, a->rows, a->dtype, stream);
+    return b200_ring_store_keep(a->k, a->ldk, a->v, a->ldv, const_cast<void*>(a->k_ring), const_cast<void*>(a->v_ring), a->ring, a->keep,
+                                a->n_kv_head * a->dk, a->n_kv_head * a->dv, a->seqs, a->row_seq, a->rows, a->dtype, stream);
   return B200_OK;
 }
 
 int b200_ring_store(const void* k, int64_t ldk, const void* v, int64_t ldv, void* k_ring, void* v_ring, int ring, int kcols, int vcols,
                     const int32_t* seqs, const int32_t* row_seq, int64_t rows, int dtype, b200_stream_t stream) {
+  return b200_ring_store_keep(k, ldk, v, ldv, k_ring, v_ring, ring, 0, kcols, vcols, seqs, row_seq, rows, dtype, stream);
+}
+
+int b200_ring_store_keep(const void* k, int64_t ldk, const void* v, int64_t ldv, void* k_ring, void* v_ring, int ring, int keep, int kcols, int vcols,
+                         const int32_t* seqs, const int32_t* row_seq, int64_t rows, int dtype, b200_stream_t stream) {
   B200_CHECK_ARG(k && v && k_ring && v_ring && seqs && row_seq, "b200_ring_store: null pointer");
-  B200_CHECK_ARG(ring > 0 && kcols > 0 && vcols > 0 && rows > 0 && rows <= 0x7fffffff, "b200_ring_store: bad shape");
+  B200_CHECK_ARG(ring > 0 && keep >= 0 && kcols > 0 && vcols > 0 && rows > 0 && rows <= 0x7fffffff, "b200_ring_store: bad shape");
   B200_CHECK_ARG((reinterpret_cast<uintptr_t>(seqs) & 15) == 0, "b200_ring_store: seqs must be 16-byte aligned");
   B200_FLOAT_TYPES(dtype, T, B200_CUDA(launch(ring_store_kernel<T>, dim3((unsigned)rows), dim3(128), 0, (cudaStream_t)stream, (const T*)k, ldk,
-                                               (const T*)v, ldv, (T*)k_ring, (T*)v_ring, ring, kcols, vcols, reinterpret_cast<const int4*>(seqs), row_seq)));
+                                               (const T*)v, ldv, (T*)k_ring, (T*)v_ring, ring, keep, kcols, vcols, reinterpret_cast<const int4*>(seqs), row_seq)));
   return B200_OK;
 }
 

@@ -605,14 +605,15 @@ def embed_pos(tokens: torch.Tensor, pos: Optional[torch.Tensor], embed: torch.Te
     return x, act
 
 
-def _seg(inp: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, d: int, plus_one: bool, in_rows=None, out_rows=None) -> "C.RmsRowsSeg":
+def _seg(inp: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, d: int, plus_one: bool, in_rows=None, out_rows=None, center: bool = False) -> "C.RmsRowsSeg":
+    """center: the row minus its mean is normed (a layer norm without bias)."""
     if inp.stride(-1) != 1 or out.stride(-1) != 1 or not weight.is_contiguous():
         raise C.B200Error("rms_rows: rows must be contiguous")
     for idx in (in_rows, out_rows):
         if idx is not None and (idx.dtype != torch.int64 or not idx.is_contiguous()):
             raise C.B200Error("rms_rows: row indices must be contiguous int64")
     return C.RmsRowsSeg(inp=inp.data_ptr(), weight=weight.data_ptr(), out=out.data_ptr(), in_rows=C.ptr(in_rows), out_rows=C.ptr(out_rows),
-                        ld_in=inp.stride(-2), ld_out=out.stride(-2), d=d, plus_one=int(plus_one))
+                        ld_in=inp.stride(-2), ld_out=out.stride(-2), d=d, plus_one=int(plus_one), center=int(center))
 
 
 def rms_rows(rows: int, eps: float, *segs: "C.RmsRowsSeg", in_dtype: torch.dtype, out_dtype: torch.dtype, device: torch.device) -> None:
@@ -661,6 +662,11 @@ def scale_f32(t: torch.Tensor, scale: float) -> torch.Tensor:
     out = torch.empty(t.shape, dtype=torch.float32, device=t.device)
     C.check(C.load_core().b200_scale_f32(t.data_ptr(), float(scale), out.data_ptr(), t.numel(), _code(t), C.stream_ptr(t.device)), "scale_f32")
     return out
+
+
+def mm_f32(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """a (n, k) @ w (m, k)^T by the vendor GEMM, accumulated and returned in fp32."""
+    return torch.mm(a, w.t()) if a.dtype == torch.float32 else torch.mm(a, w.t(), out_dtype=torch.float32)
 
 
 LATENT_PREFILL_MMA = True   # tests switch it off to reach the any-size kernel with tensor-core-sized heads
@@ -835,17 +841,20 @@ def moe_combine(y: torch.Tensor, plan: MoEPlan, wts: torch.Tensor) -> torch.Tens
 # ---------------------------------------------------------------------------------------------------------
 def sandwich_residual(x: torch.Tensor, y0: torch.Tensor, post_w: Optional[torch.Tensor], eps: float, *, w0: Optional[torch.Tensor] = None,
                       y1: Optional[torch.Tensor] = None, w1: Optional[torch.Tensor] = None, extra: Optional[torch.Tensor] = None,
-                      pre_w: Optional[torch.Tensor] = None, act: Optional[torch.Tensor] = None) -> None:
-    """x (fp32, in place) += norm(y) * post_w [+ extra]; act = T(norm(x) * pre_w).  y = y0, or with y1 the mean of the two branches
-    each normed with its weight (w0, w1)."""
-    C.require_cuda(x, y0, y1, post_w, extra, pre_w, act)
+                      pre_w: Optional[torch.Tensor] = None, act: Optional[torch.Tensor] = None, pre_center: bool = False,
+                      cast: Optional[torch.Tensor] = None) -> None:
+    """x (fp32, in place) += norm(y) * post_w [+ extra]; act = T(norm(x) * pre_w); cast = T(x).  y = y0, or with y1 the mean of the two
+    branches each normed with its weight (w0, w1).  pre_center: act norms x minus its mean (a layer norm without bias)."""
+    C.require_cuda(x, y0, y1, post_w, extra, pre_w, act, cast)
+    if cast is not None and (cast.dtype != y0.dtype or not cast.is_contiguous()):
+        raise C.B200Error("sandwich_residual: the cast must be contiguous in the branches' dtype")
     if x.dtype != torch.float32 or not x.is_contiguous() or not y0.is_contiguous() or (y1 is not None and not y1.is_contiguous()):
         raise C.B200Error("sandwich_residual: x must be contiguous fp32, the branches contiguous")
     if extra is not None and (extra.dtype != torch.float32 or not extra.is_contiguous()):
         raise C.B200Error("sandwich_residual: extra must be contiguous fp32")
     d = x.shape[-1]
     args = C.SandwichArgs(y0=y0.data_ptr(), w0=C.ptr(w0), y1=C.ptr(y1), w1=C.ptr(w1), post_w=C.ptr(post_w), extra=C.ptr(extra), pre_w=C.ptr(pre_w),
-                          x=x.data_ptr(), act=C.ptr(act), rows=x.numel() // d, d=d, eps=float(eps), dtype=_code(y0))
+                          x=x.data_ptr(), act=C.ptr(act), rows=x.numel() // d, d=d, eps=float(eps), dtype=_code(y0), pre_center=int(pre_center), cast=C.ptr(cast))
     C.check(C.load_core().b200_sandwich_residual(ctypes.byref(args), C.stream_ptr(x.device)), "sandwich_residual")
 
 
@@ -866,6 +875,18 @@ def glu(x: torch.Tensor, kind: int) -> torch.Tensor:
     ff = x.shape[-1] // 2
     out = torch.empty(x.shape[:-1] + (ff,), dtype=x.dtype, device=x.device)
     C.check(C.load_core().b200_glu(x.data_ptr(), out.data_ptr(), x.numel() // (2 * ff), ff, kind, _code(x), C.stream_ptr(x.device)), "glu")
+    return out
+
+
+def token_gate(z: torch.Tensor, tokens: torch.Tensor, table: torch.Tensor, off: int, kind: int) -> torch.Tensor:
+    """z (n, cols), tokens int32 (n,), table (vocab, columns) -> act(z) * table[tokens, off : off + cols] (n, cols)."""
+    C.require_cuda(z, tokens, table)
+    if z.dtype != table.dtype or z.stride(-1) != 1 or table.stride(-1) != 1 or tokens.dtype != torch.int32 or not tokens.is_contiguous():
+        raise C.B200Error("token_gate: projection and table in one dtype with unit inner stride, int32 tokens")
+    n, cols = z.shape
+    out = torch.empty((n, cols), dtype=z.dtype, device=z.device)
+    C.check(C.load_core().b200_token_gate(z.data_ptr(), z.stride(0), tokens.data_ptr(), table.data_ptr(), table.stride(0), off, table.shape[0], out.data_ptr(),
+                                          n, cols, kind, _code(z), C.stream_ptr(z.device)), "token_gate")
     return out
 
 
@@ -975,6 +996,44 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta_in: torch
     return out
 
 
+def linear_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, seqs: torch.Tensor, max_rows: int, heads: int, dk: int, dv: int,
+                *, silu: bool = False, q_scale: float = 1.0, head_decay: Optional[torch.Tensor] = None, decay_in: Optional[torch.Tensor] = None,
+                decay_bias: Optional[torch.Tensor] = None, tau: float = 1.0) -> torch.Tensor:
+    """Decaying linear attention over the step's rows: per head S <- diag(g) S + k v^T, o = S^T q; state (slots, heads * dk * dv) fp32 is
+    read (unless the sequence starts at 0) and written.  q, k (n, heads * dk) and v (n, heads * dv) are raw projections (`silu`: each passes
+    through it; q then times q_scale).  g: head_decay fp32 (heads,), fixed -- or decay_in fp32 (n, heads * dk), raw and used as scratch, with
+    decay_bias (heads * dk,) and tau: sigmoid(decay_in + decay_bias)^(1 / tau).  -> fp32 (n, heads * dv)"""
+    C.require_cuda(q, k, v, state, seqs, head_decay, decay_in, decay_bias)
+    if not (q.dtype == k.dtype == v.dtype) or state.dtype != torch.float32 or seqs.dtype != torch.int32 or not seqs.is_contiguous():
+        raise C.B200Error("linear_attn: q, k, v of one dtype, fp32 state, int32 seqs")
+    if (head_decay is None) == (decay_in is None):
+        raise C.B200Error("linear_attn: either fixed decays per head or per-channel decays")
+    if head_decay is not None and (head_decay.dtype != torch.float32 or head_decay.numel() != heads or not head_decay.is_contiguous()):
+        raise C.B200Error("linear_attn: head_decay must be `heads` contiguous fp32 numbers")
+    if decay_in is not None and (decay_in.dtype != torch.float32 or decay_in.stride(-1) != 1 or decay_bias is None or decay_bias.dtype != q.dtype
+                                 or decay_bias.numel() != heads * dk or not decay_bias.is_contiguous()):
+        raise C.B200Error("linear_attn: per-channel decays are fp32 rows with a bias of heads * dk numbers in the projections' dtype")
+    if any(t.stride(-1) != 1 for t in (q, k, v)) or not state.is_contiguous():
+        raise C.B200Error("linear_attn: unit inner strides, contiguous states")
+    n, lib = q.shape[0], C.load_core()
+    out = torch.empty((n, heads * dv), dtype=torch.float32, device=q.device)
+    need = lib.b200_linear_attn_workspace_bytes(n, max_rows, seqs.shape[0], heads, dk, dv)
+    ws = _ws("linear_attn", q.device, need) if need else None
+    args = C.LinearAttnArgs(q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), ldq=q.stride(0), ldk=k.stride(0), ldv=v.stride(0), act=int(silu),
+                            q_scale=float(q_scale), decay_in=C.ptr(decay_in), ld_decay=0 if decay_in is None else decay_in.stride(0),
+                            decay_bias=C.ptr(decay_bias), tau=float(tau), head_decay=C.ptr(head_decay), state=state.data_ptr(),
+                            state_slot_stride=state.stride(0), out=out.data_ptr(), ldo=out.stride(0), seqs=seqs.data_ptr(), n_seqs=seqs.shape[0],
+                            rows=n, max_rows=int(max_rows), heads=heads, dk=dk, dv=dv, dtype=_code(q), workspace=C.ptr(ws),
+                            workspace_bytes=0 if ws is None else ws.numel() * ws.element_size())
+    C.check(lib.b200_linear_attn(ctypes.byref(args), C.stream_ptr(q.device)), "linear_attn")
+    return out
+
+
+def linear_attn_tune(piece: int = 0) -> int:
+    """Test and tuning knob: tokens per piece of a prompt (0: chosen by size); returns the previous setting."""
+    return int(C.load_core().b200_linear_attn_tune(int(piece)))
+
+
 GATE_SILU, GATE_SIGMOID = 1, 2
 
 
@@ -995,12 +1054,15 @@ WINDOW_PREFILL_MMA = True   # tests switch it off to run whole prompts with tens
 def window_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_ring: torch.Tensor, v_ring: torch.Tensor, sink: Optional[torch.Tensor],
                 seqs: torch.Tensor, row_seq: torch.Tensor, max_q_len: int, n_head: int, n_kv_head: int, dk: int, dv: int, window: int,
                 scale: float, from_start: bool = False, *, dist: Optional[Tuple[torch.Tensor, torch.Tensor]] = None,
-                gate: Optional[torch.Tensor] = None, gate_per_head: bool = False) -> torch.Tensor:
+                gate: Optional[torch.Tensor] = None, gate_per_head: bool = False, keep: int = 0, softcap: float = 0.0) -> torch.Tensor:
     """Sliding-window attention with a sink over this step's k / v rows and the rings (slots, ring, G * dk | dv) of earlier
     positions; afterwards the step's rows enter the rings.  -> (n, n_head * dv).  from_start: every sequence of the step begins
     at position 0, so nothing is read from the rings -- bf16 prompts with 64- or 128-wide heads then run on the tensor-core tiles
     of the prefill kernel the other models use.  dist = (r1, r2), n_head numbers each: score -= r1 ln(1 + r2 (i - j)).  gate: raw
-    projections of the rows (n, n_head) with gate_per_head, else (n, n_head * dv); the output is multiplied by their sigmoid."""
+    projections of the rows (n, n_head) with gate_per_head, else (n, n_head * dv); the output is multiplied by their sigmoid.  keep: that
+    many first positions stay visible to every later row (the rings then hold keep + ring rows per slot); softcap: scores become
+    softcap * tanh(score / softcap) -- with either, bf16 prompts run on the tensor-core tiles for head sizes that are multiples of 8 up to
+    128, equal or not."""
     r1, r2 = dist if dist is not None else (None, None)
     C.require_cuda(q, k, v, k_ring, v_ring, sink, seqs, row_seq, r1, r2, gate)
     if dist is not None and not (r1.dtype == r2.dtype == q.dtype and r1.numel() == r2.numel() == n_head and r1.is_contiguous() and r2.is_contiguous()):
@@ -1013,10 +1075,11 @@ def window_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_ring: torch
         raise C.B200Error("window_attn: one dtype, contiguous rings")
     if q.stride(-1) != 1 or k.stride(-1) != 1 or v.stride(-1) != 1 or seqs.dtype != torch.int32 or not seqs.is_contiguous():
         raise C.B200Error("window_attn: unit inner strides, int32 seqs")
-    ring = k_ring.shape[1]
+    ring = k_ring.shape[1] - keep
     out = torch.empty((q.shape[0], n_head * dv), dtype=q.dtype, device=q.device)
     lib, st = C.load_core(), C.stream_ptr(q.device)
-    if (from_start and max_q_len > 1 and WINDOW_PREFILL_MMA and q.dtype == torch.bfloat16 and dk == dv and dk in (64, 128)
+    mma = from_start and max_q_len > 1 and WINDOW_PREFILL_MMA and q.dtype == torch.bfloat16
+    if (mma and keep == 0 and softcap == 0.0 and dk == dv and dk in (64, 128)
             and not (q.stride(0) | k.stride(0) | v.stride(0)) & 7 and not (q.data_ptr() | k.data_ptr() | v.data_ptr() | seqs.data_ptr()) & 15):
         C.check(lib.b200_attn_prefill_window_ex(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), seqs.data_ptr(),
                                                 seqs.shape[0], max_q_len, out.data_ptr(), out.stride(0), n_head, n_kv_head, dk, float(scale), window,
@@ -1028,7 +1091,14 @@ def window_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_ring: torch
     args = C.WindowAttnArgs(row_seq=row_seq.data_ptr(), rows=q.shape[0], q=q.data_ptr(), k=k.data_ptr(), v=v.data_ptr(), out=out.data_ptr(),
                             ldq=q.stride(0), ldk=k.stride(0), ldv=v.stride(0), ldo=out.stride(0), k_ring=k_ring.data_ptr(), v_ring=v_ring.data_ptr(), sink=C.ptr(sink), seqs=seqs.data_ptr(),
                             n_seqs=seqs.shape[0], max_q_len=max_q_len, ring=ring, n_head=n_head, n_kv_head=n_kv_head, dk=dk, dv=dv, window=window,
-                            scale=float(scale), dtype=_code(q), dist_r1=C.ptr(r1), dist_r2=C.ptr(r2), gate=C.ptr(gate), ldg=ldg, gate_mode=gate_mode)
+                            scale=float(scale), dtype=_code(q), dist_r1=C.ptr(r1), dist_r2=C.ptr(r2), gate=C.ptr(gate), ldg=ldg, gate_mode=gate_mode,
+                            keep=keep, softcap=float(softcap))
+    if (mma and (keep > 0 or softcap > 0.0) and dist is None and scale > 0.0 and dk % 8 == 0 and dv % 8 == 0 and dk <= 128 and dv <= 128
+            and not (q.stride(0) | k.stride(0) | v.stride(0)) & 7 and not (q.data_ptr() | k.data_ptr() | v.data_ptr() | seqs.data_ptr()) & 15):
+        C.check(lib.b200_window_attn_tiles(ctypes.byref(args), st), "window_attn_tiles")
+        C.check(lib.b200_ring_store_keep(k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), k_ring.data_ptr(), v_ring.data_ptr(), ring, keep,
+                                         n_kv_head * dk, n_kv_head * dv, seqs.data_ptr(), row_seq.data_ptr(), q.shape[0], _code(q), st), "ring_store")
+        return out
     C.check(lib.b200_window_attn(ctypes.byref(args), st), "window_attn")
     return out
 
@@ -1067,19 +1137,22 @@ def depth_residual(x_in: torch.Tensor, x_out: torch.Tensor, eps: float, groups: 
 
 def rope_seg(inp: torch.Tensor, out: torch.Tensor, heads: int, dim: int, *, norm_w: Optional[torch.Tensor] = None, freq: Optional[torch.Tensor] = None,
              rot_off: int = 0, rot_dims: int = 0, interleaved: bool = True, mag: float = 1.0, out_rows: Optional[torch.Tensor] = None,
-             in_stride: Optional[int] = None, out_stride: Optional[int] = None) -> "C.HeadRopeSeg":
+             in_stride: Optional[int] = None, out_stride: Optional[int] = None, norm_all: bool = False) -> "C.HeadRopeSeg":
     """One group of `heads` heads of `dim` numbers for ``head_rope``: `inp` / `out` are 2-d views (rows, columns) whose first column
-    is the group's first head; heads lie `in_stride` / `out_stride` (default dim) numbers apart.  freq: fp32 (rot_dims / 2,)."""
+    is the group's first head; heads lie `in_stride` / `out_stride` (default dim) numbers apart.  freq: fp32 or fp64 (rot_dims / 2,).
+    norm_all: one norm over all heads of a row, norm_w of heads * dim numbers."""
     if inp.stride(-1) != 1 or out.stride(-1) != 1 or inp.dtype != out.dtype:
         raise C.B200Error("head_rope: rows of one dtype with unit inner stride")
-    if freq is not None and (freq.dtype != torch.float32 or not freq.is_contiguous() or freq.numel() < rot_dims // 2):
-        raise C.B200Error("head_rope: frequencies must be contiguous fp32, one per rotated pair")
+    if freq is not None and (freq.dtype not in (torch.float32, torch.float64) or not freq.is_contiguous() or freq.numel() < rot_dims // 2):
+        raise C.B200Error("head_rope: frequencies must be contiguous fp32 or fp64, one per rotated pair")
+    if norm_all and (norm_w is None or norm_w.numel() != heads * dim or not norm_w.is_contiguous()):
+        raise C.B200Error("head_rope: a norm over all heads needs one contiguous weight per number of the row")
     if out_rows is not None and (out_rows.dtype != torch.int64 or not out_rows.is_contiguous()):
         raise C.B200Error("head_rope: row indices must be contiguous int64")
     return C.HeadRopeSeg(inp=inp.data_ptr(), out=out.data_ptr(), norm_w=C.ptr(norm_w), freq=C.ptr(freq) if rot_dims else None, out_rows=C.ptr(out_rows),
                          ld_in=inp.stride(-2), ld_out=out.stride(-2), heads=heads, dim=dim, in_stride=dim if in_stride is None else in_stride,
                          out_stride=dim if out_stride is None else out_stride, rot_off=rot_off, rot_dims=rot_dims, interleaved=int(interleaved),
-                         mag=float(mag))
+                         mag=float(mag), norm_all=int(norm_all), freq_f64=int(freq is not None and freq.dtype == torch.float64))
 
 
 def head_rope(rows: int, row_pos: torch.Tensor, eps: float, *segs: "C.HeadRopeSeg", dtype: torch.dtype, device: torch.device) -> None:

@@ -22,7 +22,7 @@ batches for ``generate.serve.Session``.
 """
 from __future__ import annotations
 
-from typing import Any, Dict, List, Optional, Sequence, Tuple
+from typing import Any, Dict, List, Optional, Tuple
 
 import torch
 import torch.nn as nn
@@ -32,7 +32,7 @@ from . import kernels as K
 from .config import DenseMLPSpec, GatedMoESpec, LefalixConfig, LefalixLayerSpec
 from .delta import GatedDeltaRule
 from .moe import DenseMLP, GatedSparseExperts
-from .ragged import RaggedBatch, SlotAllocator, SlotServed, state_batch
+from .ragged import RaggedBatch, StateServed
 from .window import WindowAttention
 
 
@@ -90,7 +90,8 @@ class LefalixBlock(nn.Module):
             K.sandwich_residual(x, self.mlp(act), self.norm_2b, self.eps, pre_w=next_norm, act=act)
 
 
-class Lefalix(SlotServed, nn.Module):
+class Lefalix(StateServed, nn.Module):
+    needs_positions = False    # the convolution kernel takes positions from the sequence table
     repeatable_steps = False   # a step advances recurrent states and convolution tails: repeating it is not idempotent
 
     def __init__(self, config: LefalixConfig) -> None:
@@ -101,41 +102,8 @@ class Lefalix(SlotServed, nn.Module):
         self.blocks = nn.ModuleList(LefalixBlock(config, spec) for spec in config.layers)
         self.final_norm = nn.Parameter(torch.ones(d), requires_grad=False)
         self.head = nn.Parameter(torch.empty(config.vocab_size, d), requires_grad=False)
-        self.runs = config.schedule()                       # (layer, state index, the embedding re-enters before this run)
-        self._max_seq_length = config.block_size
-        self.slots: Optional[SlotAllocator] = None
-        self.states: Optional[nn.ModuleList] = None         # one state per layer RUN: a repeated layer has one per repetition
+        self.init_serving(config.schedule())                # runs: (layer, state index, the embedding re-enters before this run)
         self.trace: Optional[List[torch.Tensor]] = None     # debugging: set to a list to receive the stream after every layer run
-
-    # ---- the surface generate() uses (with ``SlotServed``) --------------------------------------------------------
-    def set_kv_cache(self, batch_size: int, rope_cache_length: Optional[int] = None, device: Optional[torch.device] = None,
-                     dtype: Optional[torch.dtype] = None) -> None:
-        """`batch_size` state slots for every layer run.  A state is constant in size: nothing depends on `max_seq_length`."""
-        device = device if device is not None else self.device
-        dtype = dtype if dtype is not None else self.dtype
-        self.states = nn.ModuleList(self.blocks[layer].mixer.build_state(batch_size, device, dtype) for layer, _, _ in self.runs)
-        self.slots = SlotAllocator(batch_size)
-        self._drop_graphs()
-
-    def clear_kv_cache(self) -> None:
-        self.states = None
-        self.slots = None
-        self._drop_graphs()
-
-    def reset_caches(self) -> None:
-        for t in self.state_tensors():
-            t.zero_()
-
-    def state_tensors(self) -> List[torch.Tensor]:
-        return [t for st in (self.states or []) for t in st.tensors()]
-
-    def _apply(self, fn, recurse: bool = True):
-        self._drop_graphs()
-        states, self.states = self.states, None     # states keep their own dtypes (fp32 matrices): a cast of the model skips them
-        try:
-            return super()._apply(fn, recurse)
-        finally:
-            self.states = states
 
     # ---- weights ----------------------------------------------------------------------------------------------------
     def reset_parameters(self, seed: int = 1234, std: float = 0.02) -> None:
@@ -254,51 +222,3 @@ class Lefalix(SlotServed, nn.Module):
             K.rms_rows(rows, eps, K.rms_seg(x, self.final_norm, xn, d, False, in_rows=want_rows), in_dtype=torch.float32, out_dtype=self.dtype,
                        device=x.device)
             return K.scale_f32(F.linear(xn, self.head), 1.0)
-
-    @torch.inference_mode()
-    def step(self, tokens: Sequence[int], seqs: Sequence[Tuple[int, int, int]], want: Optional[Sequence[int]] = None) -> torch.Tensor:
-        """One step over a ragged batch.  `tokens`: the new tokens of all sequences, sequence after sequence; `seqs`: per
-        sequence (state slot, position of its first new token, number of new tokens); `want`: indices into `tokens` of the rows
-        whose logits are returned (default: all).  Returns fp32 (rows, vocab).  A sequence at position 0 starts from an empty
-        state whatever its slot held; otherwise its slot must hold the state its earlier tokens left."""
-        if self.slots is None:
-            raise TypeError("You need to call `set_kv_cache()` first")
-        dev = self.device
-        n = len(tokens)
-        if n == 0 or n != sum(s[2] for s in seqs):
-            raise ValueError("step: the sequence lengths must add up to the number of tokens (> 0)")
-        for slot, start, length in seqs:
-            if not 0 <= slot < self.slots.capacity or length <= 0 or start < 0 or start + length > self.max_seq_length:
-                raise ValueError(f"step: sequence (slot {slot}, start {start}, length {length}) does not fit {self.slots.capacity} slots")
-        batch, toks = state_batch(seqs, dev, tokens)
-        want_rows = None if want is None else torch.tensor(list(want), dtype=torch.int64).to(dev, non_blocking=True)
-        return self._run(toks, batch, want_rows)
-
-    def forward(self, idx: torch.Tensor, input_pos: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """idx (B, T) token ids, batch row b = state slot b, all rows at the positions `input_pos` (T,), as ``GPT.forward``.
-        Returns fp32 logits (B, T, vocab).  T = 1 runs without any host synchronisation (CUDA-graph capturable)."""
-        B, T = idx.shape
-        if input_pos is None:
-            raise TypeError("Lefalix runs over its states: pass input_pos")
-        if self.slots is None:
-            raise TypeError("You need to call `set_kv_cache()` first")
-        if B > self.slots.capacity:
-            raise ValueError(f"batch of {B} rows, but only {self.slots.capacity} state slots")
-        dev = idx.device
-        const = self.__dict__.get("_const")
-        if const is None or const[0].numel() < B or const[0].device != dev:
-            slots = torch.arange(max(B, self.slots.capacity), dtype=torch.int32, device=dev)
-            const = self.__dict__["_const"] = (slots, torch.ones_like(slots))
-        ar = const[0][:B]
-        if T == 1:
-            seq_state = torch.stack([ar, const[1][:B], input_pos.to(torch.int32).expand(B), ar], dim=1).contiguous()
-            batch = RaggedBatch(row_pos=None, row_slot=None, cache_rows=None, decode=True, context_hint=self.max_seq_length, seq_state=seq_state,
-                                row_seq=ar)
-            return self._run(idx.reshape(B).to(torch.int32), batch, None).view(B, 1, -1)
-        start = int(input_pos[0])   # host read: the prompt's rows are laid out on the host
-        if start + T > self.max_seq_length:
-            raise ValueError(f"Cannot forward sequence of length {start + T}, max seq length is only {self.max_seq_length}.")
-        seq_state = torch.tensor([(b * T, T, start, b) for b in range(B)], dtype=torch.int32).to(dev)
-        batch = RaggedBatch(row_pos=None, row_slot=None, cache_rows=None, decode=False, context_hint=start + T, max_q_len=T, seq_state=seq_state,
-                            identity_ctx=start == 0, row_seq=ar.repeat_interleave(T))
-        return self._run(idx.reshape(B * T).to(torch.int32), batch, None).view(B, T, -1)

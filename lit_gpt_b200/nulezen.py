@@ -15,12 +15,12 @@ to the vendor GEMM, everything else is this library's kernels: ``K.scaled_residu
 block's norm in one elementwise launch (the norm needs no statistics).
 
 Sequences live in slots: per layer run and slot the key / value rings of one window, so a sequence can be any length.  The model plugs
-into the entry points the other slot-served models use: ``forward(idx, input_pos)`` for ``generate.base`` (single-token steps are
-CUDA-graph capturable) and ``step`` over ragged batches for ``generate.serve.Session``.
+into the entry points the other slot-served models use (``ragged.StateServed``): ``forward(idx, input_pos)`` for ``generate.base``
+(single-token steps are CUDA-graph capturable) and ``step`` over ragged batches for ``generate.serve.Session``.
 """
 from __future__ import annotations
 
-from typing import Dict, List, Optional, Sequence, Tuple
+from typing import Dict, List, Optional, Tuple
 
 import torch
 import torch.nn as nn
@@ -28,7 +28,7 @@ import torch.nn as nn
 from . import kernels as K
 from .config import ClampedMoESpec, DenseMLPSpec, NulezenConfig, NulezenLayerSpec
 from .moe import ClampedSparseExperts, DenseMLP
-from .ragged import RaggedBatch, SlotAllocator, SlotServed, state_batch
+from .ragged import RaggedBatch, StateServed
 from .window import GatedWindowAttention
 
 
@@ -71,7 +71,7 @@ class NulezenBlock(nn.Module):
                           act=act)
 
 
-class Nulezen(SlotServed, nn.Module):
+class Nulezen(StateServed, nn.Module):
 
     def __init__(self, config: NulezenConfig) -> None:
         super().__init__()
@@ -85,41 +85,12 @@ class Nulezen(SlotServed, nn.Module):
             self.loop_in_x = nn.Parameter(torch.empty(d, d), requires_grad=False)
             self.loop_in_e = nn.Parameter(torch.empty(d, d), requires_grad=False)
             self.loop_step = nn.Parameter(torch.zeros(config.loop_times, d), requires_grad=False)
-        self.runs = config.schedule()                       # (layer, state index, pass this run opens or -1)
-        self._max_seq_length = config.block_size
-        self.slots: Optional[SlotAllocator] = None
-        self.states: Optional[nn.ModuleList] = None         # one state per layer RUN: a repeated layer has one per repetition
+        self.init_serving(config.schedule())                # runs: (layer, state index, pass this run opens or -1)
         self.trace: Optional[List[torch.Tensor]] = None     # debugging: set to a list to receive the stream after every layer run
 
     @property
     def head(self) -> torch.Tensor:
         return self.embed
-
-    # ---- the surface generate() uses (with ``SlotServed``) --------------------------------------------------------
-    def set_kv_cache(self, batch_size: int, rope_cache_length: Optional[int] = None, device: Optional[torch.device] = None,
-                     dtype: Optional[torch.dtype] = None) -> None:
-        """`batch_size` state slots for every layer run.  A state is constant in size: nothing depends on `max_seq_length`."""
-        device = device if device is not None else self.device
-        dtype = dtype if dtype is not None else self.dtype
-        self.states = nn.ModuleList(self.blocks[layer].mixer.build_state(batch_size, device, dtype) for layer, _, _ in self.runs)
-        self.slots = SlotAllocator(batch_size)
-        self._drop_graphs()
-
-    def clear_kv_cache(self) -> None:
-        self.states = None
-        self.slots = None
-        self._drop_graphs()
-
-    def reset_caches(self) -> None:
-        for t in self.state_tensors():
-            t.zero_()
-
-    def state_tensors(self) -> List[torch.Tensor]:
-        return [t for st in (self.states or []) for t in st.tensors()]
-
-    def _apply(self, fn, recurse: bool = True):
-        self._drop_graphs()
-        return super()._apply(fn, recurse)
 
     # ---- weights ----------------------------------------------------------------------------------------------------
     def reset_parameters(self, seed: int = 1234, std: float = 0.02) -> None:
@@ -214,10 +185,6 @@ class Nulezen(SlotServed, nn.Module):
             raise KeyError(f"unexpected tensors in the checkpoint: {extra[:6]}")
 
     # ---- one step ---------------------------------------------------------------------------------------------------
-    def _mm(self, a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
-        """a (n, k) @ w (m, k)^T accumulated and returned in fp32"""
-        return torch.mm(a, w.t()) if a.dtype == torch.float32 else torch.mm(a, w.t(), out_dtype=torch.float32)
-
     def _run(self, tokens: torch.Tensor, batch: RaggedBatch, want_rows: Optional[torch.Tensor]) -> torch.Tensor:
         """tokens int32 (n,) -> fp32 logits (rows wanted or n, vocab)"""
         c = self.config
@@ -226,13 +193,13 @@ class Nulezen(SlotServed, nn.Module):
             x, emb = K.embed_pos(tokens, None, self.embed, None, c.embedding_scale)     # the stream and the embedding in the product dtype
             act = torch.empty_like(emb)
             cast = emb                                            # the stream in the product dtype, where a pass's entry reads it
-            from_emb = self._mm(emb, self.loop_in_e) if c.looped else None     # the embedding's share of every pass's entry
+            from_emb = K.mm_f32(emb, self.loop_in_e) if c.looped else None     # the embedding's share of every pass's entry
             if not runs or runs[0][2] < 0:
                 K.scaled_residual(x, norm=(self.blocks[runs[0][0]].norm if runs else self.final_norm).terms(), act=act)
             for r, (layer, state, opens) in enumerate(runs):
                 block = self.blocks[layer]
                 if opens >= 0:   # x <- W_in [x ; x0] + step[t], then this block's norm
-                    x = self._mm(cast, self.loop_in_x)
+                    x = K.mm_f32(cast, self.loop_in_x)
                     K.scaled_residual(x, extra=from_emb, row_add=self.loop_step[opens], norm=block.norm.terms(), act=act)
                 nxt, cast_out = None, None
                 if r + 1 < len(runs):
@@ -246,53 +213,4 @@ class Nulezen(SlotServed, nn.Module):
             xw = x if want_rows is None else K.gather_rows(x, want_rows)
             xn = torch.empty(xw.shape, dtype=self.dtype, device=x.device)
             K.scaled_residual(xw, norm=self.final_norm.terms(), act=xn)
-            return K.scale_f32(self._mm(xn, self.embed), c.logit_scale)
-
-    @torch.inference_mode()
-    def step(self, tokens: Sequence[int], seqs: Sequence[Tuple[int, int, int]], want: Optional[Sequence[int]] = None) -> torch.Tensor:
-        """One step over a ragged batch.  `tokens`: the new tokens of all sequences, sequence after sequence; `seqs`: per
-        sequence (state slot, position of its first new token, number of new tokens); `want`: indices into `tokens` of the rows
-        whose logits are returned (default: all).  Returns fp32 (rows, vocab).  A sequence's slot must hold the rings its earlier
-        tokens left; a reused slot needs no clearing, since only a sequence's own positions are ever read."""
-        if self.slots is None:
-            raise TypeError("You need to call `set_kv_cache()` first")
-        dev = self.device
-        n = len(tokens)
-        if n == 0 or n != sum(s[2] for s in seqs):
-            raise ValueError("step: the sequence lengths must add up to the number of tokens (> 0)")
-        for slot, start, length in seqs:
-            if not 0 <= slot < self.slots.capacity or length <= 0 or start < 0 or start + length > self.max_seq_length:
-                raise ValueError(f"step: sequence (slot {slot}, start {start}, length {length}) does not fit {self.slots.capacity} slots")
-        batch, toks = state_batch(seqs, dev, tokens, positions=True)
-        want_rows = None if want is None else torch.tensor(list(want), dtype=torch.int64).to(dev, non_blocking=True)
-        return self._run(toks, batch, want_rows)
-
-    def forward(self, idx: torch.Tensor, input_pos: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """idx (B, T) token ids, batch row b = state slot b, all rows at the positions `input_pos` (T,), as ``GPT.forward``.
-        Returns fp32 logits (B, T, vocab).  T = 1 runs without any host synchronisation (CUDA-graph capturable)."""
-        B, T = idx.shape
-        if input_pos is None:
-            raise TypeError("Nulezen runs over its states: pass input_pos")
-        if self.slots is None:
-            raise TypeError("You need to call `set_kv_cache()` first")
-        if B > self.slots.capacity:
-            raise ValueError(f"batch of {B} rows, but only {self.slots.capacity} state slots")
-        dev = idx.device
-        const = self.__dict__.get("_const")
-        if const is None or const[0].numel() < B or const[0].device != dev:
-            slots = torch.arange(max(B, self.slots.capacity), dtype=torch.int32, device=dev)
-            const = self.__dict__["_const"] = (slots, torch.ones_like(slots))
-        ar = const[0][:B]
-        pos32 = input_pos.to(torch.int32)
-        if T == 1:
-            seq_state = torch.stack([ar, const[1][:B], pos32.expand(B), ar], dim=1).contiguous()
-            batch = RaggedBatch(row_pos=pos32.expand(B).contiguous(), row_slot=None, cache_rows=None, decode=True, context_hint=self.max_seq_length,
-                                seq_state=seq_state, row_seq=ar)
-            return self._run(idx.reshape(B).to(torch.int32), batch, None).view(B, 1, -1)
-        start = int(input_pos[0])   # host read: the prompt's rows are laid out on the host
-        if start + T > self.max_seq_length:
-            raise ValueError(f"Cannot forward sequence of length {start + T}, max seq length is only {self.max_seq_length}.")
-        seq_state = torch.tensor([(b * T, T, start, b) for b in range(B)], dtype=torch.int32).to(dev)
-        batch = RaggedBatch(row_pos=pos32.repeat(B), row_slot=None, cache_rows=None, decode=False, context_hint=start + T, max_q_len=T,
-                            seq_state=seq_state, identity_ctx=start == 0, row_seq=ar.repeat_interleave(T))
-        return self._run(idx.reshape(B * T).to(torch.int32), batch, None).view(B, T, -1)
+            return K.scale_f32(K.mm_f32(xn, self.embed), c.logit_scale)

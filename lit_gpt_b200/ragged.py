@@ -8,6 +8,7 @@ from dataclasses import dataclass
 from typing import Iterator, List, Optional, Sequence, Tuple
 
 import torch
+import torch.nn as nn
 
 
 @dataclass
@@ -130,3 +131,98 @@ class SlotServed:
             yield
         finally:
             torch.backends.cuda.matmul.allow_tf32 = old
+
+
+class StateServed(SlotServed):
+    """A slot-served model whose layers keep a state of constant size per slot (rings of one window, convolution tails, state matrices):
+    the states, ``step`` over ragged batches and ``forward`` for ``generate.base``.  The model calls ``init_serving(runs)`` with its layer
+    runs -- (layer index, state index, ...) in order, every run with a state of its own -- and provides ``blocks`` (whose ``mixer`` has
+    ``build_state``), ``head`` and ``_run(tokens, batch, want_rows)``."""
+
+    needs_positions = True           # the rows' positions are part of the step's description
+
+    def init_serving(self, runs: Sequence[Tuple]) -> None:
+        self.runs = list(runs)
+        self._max_seq_length = self.config.block_size
+        self.slots: Optional[SlotAllocator] = None
+        self.states: Optional[nn.ModuleList] = None   # one state per layer RUN: a repeated layer has one per repetition
+
+    def set_kv_cache(self, batch_size: int, rope_cache_length: Optional[int] = None, device: Optional[torch.device] = None,
+                     dtype: Optional[torch.dtype] = None) -> None:
+        """`batch_size` state slots for every layer run.  A state is constant in size: nothing depends on `max_seq_length`."""
+        device = device if device is not None else self.device
+        dtype = dtype if dtype is not None else self.dtype
+        self.states = nn.ModuleList(self.blocks[run[0]].mixer.build_state(batch_size, device, dtype) for run in self.runs)
+        self.slots = SlotAllocator(batch_size)
+        self._drop_graphs()
+
+    def clear_kv_cache(self) -> None:
+        self.states = None
+        self.slots = None
+        self._drop_graphs()
+
+    def reset_caches(self) -> None:
+        for t in self.state_tensors():
+            t.zero_()
+
+    def state_tensors(self) -> List[torch.Tensor]:
+        return [t for st in (self.states or []) for t in st.tensors()]
+
+    def _apply(self, fn, recurse: bool = True):
+        self._drop_graphs()
+        if self.repeatable_steps:
+            return super()._apply(fn, recurse)
+        states, self.states = self.states, None     # recurrent states keep their own dtypes (fp32 matrices): a cast of the model skips them
+        try:
+            return super()._apply(fn, recurse)
+        finally:
+            self.states = states
+
+    @torch.inference_mode()
+    def step(self, tokens: Sequence[int], seqs: Sequence[Tuple[int, int, int]], want: Optional[Sequence[int]] = None) -> torch.Tensor:
+        """One step over a ragged batch.  `tokens`: the new tokens of all sequences, sequence after sequence; `seqs`: per
+        sequence (state slot, position of its first new token, number of new tokens); `want`: indices into `tokens` of the rows
+        whose logits are returned (default: all).  Returns fp32 (rows, vocab).  A sequence at position 0 starts from an empty
+        state whatever its slot held; otherwise its slot must hold the state its earlier tokens left."""
+        if self.slots is None:
+            raise TypeError("You need to call `set_kv_cache()` first")
+        dev = self.device
+        n = len(tokens)
+        if n == 0 or n != sum(s[2] for s in seqs):
+            raise ValueError("step: the sequence lengths must add up to the number of tokens (> 0)")
+        for slot, start, length in seqs:
+            if not 0 <= slot < self.slots.capacity or length <= 0 or start < 0 or start + length > self.max_seq_length:
+                raise ValueError(f"step: sequence (slot {slot}, start {start}, length {length}) does not fit {self.slots.capacity} slots")
+        batch, toks = state_batch(seqs, dev, tokens, positions=self.needs_positions)
+        want_rows = None if want is None else torch.tensor(list(want), dtype=torch.int64).to(dev, non_blocking=True)
+        return self._run(toks, batch, want_rows)
+
+    def forward(self, idx: torch.Tensor, input_pos: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """idx (B, T) token ids, batch row b = state slot b, all rows at the positions `input_pos` (T,), as ``GPT.forward``.
+        Returns fp32 logits (B, T, vocab).  T = 1 runs without any host synchronisation (CUDA-graph capturable)."""
+        B, T = idx.shape
+        if input_pos is None:
+            raise TypeError(f"{type(self).__name__} runs over its states: pass input_pos")
+        if self.slots is None:
+            raise TypeError("You need to call `set_kv_cache()` first")
+        if B > self.slots.capacity:
+            raise ValueError(f"batch of {B} rows, but only {self.slots.capacity} state slots")
+        dev = idx.device
+        const = self.__dict__.get("_const")
+        if const is None or const[0].numel() < B or const[0].device != dev:
+            slots = torch.arange(max(B, self.slots.capacity), dtype=torch.int32, device=dev)
+            const = self.__dict__["_const"] = (slots, torch.ones_like(slots))
+        ar = const[0][:B]
+        pos32 = input_pos.to(torch.int32)
+        if T == 1:
+            seq_state = torch.stack([ar, const[1][:B], pos32.expand(B), ar], dim=1).contiguous()
+            batch = RaggedBatch(row_pos=pos32.expand(B).contiguous() if self.needs_positions else None, row_slot=None, cache_rows=None, decode=True,
+                                context_hint=self.max_seq_length, seq_state=seq_state, row_seq=ar)
+            return self._run(idx.reshape(B).to(torch.int32), batch, None).view(B, 1, -1)
+        start = int(input_pos[0])   # host read: the prompt's rows are laid out on the host
+        if start + T > self.max_seq_length:
+            raise ValueError(f"Cannot forward sequence of length {start + T}, max seq length is only {self.max_seq_length}.")
+        seq_state = torch.tensor([(b * T, T, start, b) for b in range(B)], dtype=torch.int32).to(dev)
+        batch = RaggedBatch(row_pos=pos32.repeat(B) if self.needs_positions else None, row_slot=None, cache_rows=None, decode=False,
+                            context_hint=start + T, max_q_len=T, seq_state=seq_state, identity_ctx=start == 0, row_seq=ar.repeat_interleave(T))
+        return self._run(idx.reshape(B * T).to(torch.int32), batch, None).view(B, T, -1)

@@ -15,7 +15,10 @@ library's kernels.
     s_ij   -= r1_h ln(1 + r2_h (i - j))                      (optional distance bias, two learned numbers per head)
     out     = W_o (concat_h(sum_j p_ij v_j) * sigmoid(W_g h))  (gate per output number, or one per head)
 
-optional biases on q, k, v and optional rotary positions on half-split pairs (``K.head_rope``).
+optional biases on q, k, v, optional rotary positions on half-split pairs (``K.head_rope``), and further options of
+``GatedWindowSpec``: RMS norms over all query heads and over all key heads before the rotation (same launch), capped scores
+s <- c tanh(s / c), the sink above, and kept first tokens: positions j < keep stay visible whatever the window, in cache rows of their
+own ahead of the ring's.
 """
 from __future__ import annotations
 
@@ -97,46 +100,53 @@ class WindowAttention(nn.Module):
 
 
 class RingState(nn.Module):
-    """Per slot: key / value rings (ring, kv_heads * dim | vdim) of a sequence's last `ring` positions."""
+    """Per slot: keys and values (keep + ring, kv_heads * dim | vdim) of a sequence's first `keep` and last `ring` positions."""
 
-    def __init__(self, slots: int, ring: int, k_cols: int, v_cols: int, device=None, dtype=None) -> None:
+    def __init__(self, slots: int, ring: int, k_cols: int, v_cols: int, device=None, dtype=None, keep: int = 0) -> None:
         super().__init__()
-        self.ring = ring
-        self.register_buffer("k_ring", torch.zeros((slots, ring, k_cols), device=device, dtype=dtype), persistent=False)
-        self.register_buffer("v_ring", torch.zeros((slots, ring, v_cols), device=device, dtype=dtype), persistent=False)
+        self.ring, self.keep = ring, keep
+        self.register_buffer("k_ring", torch.zeros((slots, keep + ring, k_cols), device=device, dtype=dtype), persistent=False)
+        self.register_buffer("v_ring", torch.zeros((slots, keep + ring, v_cols), device=device, dtype=dtype), persistent=False)
 
     def tensors(self):
         return [self.k_ring, self.v_ring]
 
 
 class GatedWindowAttention(nn.Module):
-    def __init__(self, width: int, spec: GatedWindowSpec, eps: float = 0.0) -> None:
+    def __init__(self, width: int, spec: GatedWindowSpec, eps: float = 0.0, align: int = 1) -> None:
+        """align: the fused projection gets zero rows at its end up to a multiple of `align` (rows of its result then start on 16-byte
+        boundaries whatever the number of heads)."""
         super().__init__()
         self.spec, self.eps, self.width = spec, eps, width
         H, G, dk, dv = spec.heads, spec.kv_heads, spec.dim, spec.vdim
         self.gate_cols = 0 if spec.gate is None else (H if spec.gate == "head" else H * dv)
         self.cols = H * dk + G * dk + G * dv + self.gate_cols
-        # fused projection: rows [0, H dk) queries, then G dk keys, G dv values, then the gate's rows
+        self.cols += -self.cols % align
+        # fused projection: rows [0, H dk) queries, then G dk keys, G dv values, then the gate's rows (and padding)
         self.w_in = nn.Parameter(torch.empty(self.cols, width), requires_grad=False)
         self.b_in = nn.Parameter(torch.zeros(self.cols), requires_grad=False) if spec.bias else None
         self.r1 = nn.Parameter(torch.zeros(H), requires_grad=False) if spec.distance else None
         self.r2 = nn.Parameter(torch.zeros(H), requires_grad=False) if spec.distance else None
+        self.q_norm = nn.Parameter(torch.ones(H * dk), requires_grad=False) if spec.qk_norm else None
+        self.k_norm = nn.Parameter(torch.ones(G * dk), requires_grad=False) if spec.qk_norm else None
+        self.sink = nn.Parameter(torch.zeros(H), requires_grad=False) if spec.sink else None
         self.w_o = nn.Parameter(torch.empty(width, H * dv), requires_grad=False)
         self._freq_cache: dict = {}
 
     def freq(self, device: torch.device) -> Optional[torch.Tensor]:
-        """Angular frequencies of the rotated pairs on `device` (fp32; made from the specification, so no cast of the module touches them)."""
+        """Angular frequencies of the rotated pairs on `device` (fp64: the kernel reduces position * frequency before the fp32 sine; made from
+        the specification, so no cast of the module touches them)."""
         rot = self.spec.rot
         if rot is None or rot.dims == 0:
             return None
         t = self._freq_cache.get(device)
         if t is None:
-            t = self._freq_cache[device] = torch.tensor(rot.frequencies(), dtype=torch.float32, device=device)
+            t = self._freq_cache[device] = torch.tensor(rot.frequencies(), dtype=torch.float64, device=device)
         return t
 
     def build_state(self, slots: int, device=None, dtype=None) -> RingState:
         s = self.spec
-        return RingState(slots, s.window, s.kv_heads * s.dim, s.kv_heads * s.vdim, device, dtype)
+        return RingState(slots, s.window, s.kv_heads * s.dim, s.kv_heads * s.vdim, device, dtype, keep=s.keep)
 
     def forward(self, h: torch.Tensor, batch: RaggedBatch, state: RingState) -> torch.Tensor:
         """h (n, width) in the matrix-product dtype -> (n, width)"""
@@ -144,15 +154,14 @@ class GatedWindowAttention(nn.Module):
         H, G, dk, dv = s.heads, s.kv_heads, s.dim, s.vdim
         proj = F.linear(h, self.w_in, self.b_in)
         q, k, v = proj[:, : H * dk], proj[:, H * dk : (H + G) * dk], proj[:, (H + G) * dk : (H + G) * dk + G * dv]
-        gate = proj[:, (H + G) * dk + G * dv :] if self.gate_cols else None
+        off = (H + G) * dk + G * dv
+        gate = proj[:, off : off + self.gate_cols] if self.gate_cols else None
         fr = self.freq(h.device)
-        if fr is not None:
-            rot = s.rot
-            K.head_rope(n, batch.row_pos, self.eps,
-                        K.rope_seg(q, q, H, dk, freq=fr, rot_dims=rot.dims, interleaved=rot.interleaved, mag=rot.magnitude),
-                        K.rope_seg(k, k, G, dk, freq=fr, rot_dims=rot.dims, interleaved=rot.interleaved, mag=rot.magnitude),
-                        dtype=h.dtype, device=h.device)
-        y = K.window_attn(q, k, v, state.k_ring, state.v_ring, None, batch.seq_state, batch.row_seq, batch.max_q_len, H, G, dk, dv, s.window,
+        if fr is not None or s.qk_norm:   # both norms and both rotations in place, one launch
+            turn = dict(freq=fr, rot_dims=s.rot.dims, interleaved=s.rot.interleaved, mag=s.rot.magnitude) if fr is not None else {}
+            K.head_rope(n, batch.row_pos, self.eps, K.rope_seg(q, q, H, dk, norm_w=self.q_norm, norm_all=s.qk_norm, **turn),
+                        K.rope_seg(k, k, G, dk, norm_w=self.k_norm, norm_all=s.qk_norm, **turn), dtype=h.dtype, device=h.device)
+        y = K.window_attn(q, k, v, state.k_ring, state.v_ring, self.sink, batch.seq_state, batch.row_seq, batch.max_q_len, H, G, dk, dv, s.window,
                           s.scale, from_start=batch.identity_ctx, dist=(self.r1, self.r2) if s.distance else None, gate=gate,
-                          gate_per_head=s.gate == "head")
+                          gate_per_head=s.gate == "head", keep=s.keep, softcap=s.softcap)
         return F.linear(y, self.w_o)

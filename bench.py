@@ -1099,6 +1099,172 @@ def run_fizadra_compare(args) -> None:
                       "gpu_launches": int(K.launch_count() - launches0), "sizes": out}), flush=True)
 
 
+# ---------------------------------------------------------------------------------------------------------
+# --compare votavik: the Votavik design beside the closest existing model (Lefalix: the other design with windowed attention behind a
+# sink and recurrent layers over an fp32 residual stream) at equal width, heads, head size, window, layers and dense feed-forward size;
+# single kernels also beside Nulezen's where that design has the nearer one.  Random weights.
+# ---------------------------------------------------------------------------------------------------------
+def run_votavik_compare(args) -> None:
+    from lit_gpt_b200 import kernels as K
+    from lit_gpt_b200.config import (ClampedGLUSpec, DeltaMixerSpec, DenseMLPSpec, GatedWindowSpec, LefalixConfig, LefalixLayerSpec, LinearMixerSpec,
+                                     ParallelMixerSpec, RotarySpec, VotavikConfig, VotavikLayerSpec, WindowMixerSpec)
+    from lit_gpt_b200.lefalix import Lefalix
+    from lit_gpt_b200.ragged import state_batch
+    from lit_gpt_b200.votavik import Votavik
+
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    peaks, peak_source = measured_peaks()
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    flush = torch.zeros(256 << 20, dtype=torch.uint8, device=dev)
+    vocab, T, side, keep, cap = 32000, args.prompt, 256, 4, 30.0
+    iters = max(3, min(args.steps, 20))
+    launches0 = K.launch_count()
+    bf = torch.bfloat16
+    out = {}
+    for name in (args.sizes.split(",") if args.sizes else LEFALIX_SIZES):
+        d, H, G, hs, W, rank, _, _, _, dff = LEFALIX_SIZES[name]
+        ff = 2 * dff // 3 // 128 * 128        # three matrices of this size hold what Lefalix's two of dff hold
+        half = RotarySpec(dims=hs // 2, base=1e6, interleaved=False)
+        att = lambda: VotavikLayerSpec("attention", GatedWindowSpec(H, G, hs, hs, W, hs ** -0.5, rot=half, gate="head", qk_norm=True, softcap=cap, keep=keep,   # noqa: E731
+                                                                    sink=True), ClampedGLUSpec(ff, 7.0))
+        lig = lambda: VotavikLayerSpec("lightning", LinearMixerSpec(H // 2, hs, hs, decay=[1 - 2.0 ** -(5 + j % 8) for j in range(H // 2)]), ClampedGLUSpec(ff, 7.0))   # noqa: E731
+        gla = lambda: VotavikLayerSpec("gla", LinearMixerSpec(H // 2, hs, hs, tau=16.0, decay_rank=rank), ClampedGLUSpec(ff, 7.0))   # noqa: E731
+        vot = Votavik(VotavikConfig(vocab_size=vocab, n_embd=d, side_dim=side, layers=[att(), lig(), gla(), att()])).to(dev).to(bf).eval()
+        vot.reset_parameters()
+        vot.max_seq_length = T + 64
+        rot = RotarySpec(dims=hs // 2, base=1e6, factor=4.0, original=4096.0, fast=32.0, slow=1.0)
+        par = lambda: LefalixLayerSpec("parallel", ParallelMixerSpec(WindowMixerSpec(H, G, hs, hs, 4, W, hs ** -0.5, rot), DeltaMixerSpec(H // 2, H // 4, hs, hs, 4)),   # noqa: E731
+                                       DenseMLPSpec(dff))
+        chd = lambda: LefalixLayerSpec("channel_delta", DeltaMixerSpec(H // 2, H // 4, hs, hs, 4, True, rank, rank), DenseMLPSpec(dff))   # noqa: E731
+        lef = Lefalix(LefalixConfig(vocab_size=vocab, n_embd=d, layers=[par(), chd(), chd(), par()])).to(dev).to(bf).eval()
+        lef.reset_parameters()
+        lef.max_seq_length = T + 64
+        res = {}
+        with torch.inference_mode():
+            for label, model in (("votavik", vot), ("lefalix", lef)):
+                for B in (1, 8):
+                    model.set_kv_cache(batch_size=B)
+                    idx = torch.randint(0, vocab, (B, T), device=dev)
+                    pos = torch.arange(T, device=dev)
+                    if B == 1:
+                        ms = _timed(lambda: model(idx, pos), iters, flush)
+                        res[f"{label}_prefill_tok_s"] = round(T / ms * 1e3)
+                    else:
+                        model(idx, pos)
+                    tok, p1 = idx[:, :1].contiguous(), torch.tensor([T], device=dev)
+                    step, graphed = _graphed(lambda: model(tok, p1))
+                    ms = _timed(step, iters, flush)
+                    res[f"{label}_decode_b{B}_tok_s"] = round(B / ms * 1e3)
+                    res[f"{label}_decode_b{B}_graphed"] = graphed
+                    del step
+                model.clear_kv_cache()
+            kern = {}
+
+            def put(key, fn, *, nbytes=None, flops=None, n=iters, **extra):
+                ms = _timed(fn, n, flush)
+                kern[key] = {"ms": ms, **extra}
+                if flops is not None:
+                    kern[key]["frac_of_measured_bf16"] = flops / (ms * 1e-3) / tf
+                if nbytes is not None:
+                    kern[key]["frac_of_measured_hbm"] = nbytes / (ms * 1e-3) / hbm
+
+            batch, _ = state_batch([(0, 0, T)], dev, positions=True)
+            B = 8
+            bd, _ = state_batch([(b, T, 1) for b in range(B)], dev, positions=True)
+            # windowed attention: the window's work is sum_i min(i + 1, W) score pairs (plus the kept tokens once they have left it)
+            q, kv = torch.randn(T, H * hs, device=dev, dtype=bf), torch.randn(T, 2 * G * hs, device=dev, dtype=bf)
+            kk, vv = kv[:, : G * hs], kv[:, G * hs :]
+            sink, gate_h = torch.zeros(H, device=dev, dtype=bf), torch.randn(T, H, device=dev, dtype=bf)
+            gate_e = torch.randn(T, H * hs, device=dev, dtype=bf)
+            r1, r2 = torch.full((H,), 0.5, device=dev, dtype=bf), torch.ones(H, device=dev, dtype=bf)
+            rings = {kp: [torch.randn(B, W + kp, G * hs, device=dev, dtype=bf) for _ in range(2)] for kp in (0, keep)}
+
+            def win(b, rows, n_rows, kp, softcap, **kw):
+                return K.window_attn(q[:rows], kk[:rows], vv[:rows], *rings[kp], kw.pop("sink", None), b.seq_state, b.row_seq, n_rows, H, G, hs, hs, W, hs ** -0.5,
+                                     from_start=n_rows > 1, keep=kp, softcap=softcap, **kw)
+
+            cases = (("votavik_kept_cap_sink_gate_per_head", keep, cap, dict(sink=sink, gate=gate_h, gate_per_head=True)), ("lefalix_sink", 0, 0.0, dict(sink=sink)),
+                     ("nulezen_distance_bias_gate_per_number", 0, 0.0, dict(dist=(r1, r2), gate=gate_e)))
+            for label, kp, sc, kw in cases:
+                pairs = sum(min(i + 1, W + kp) for i in range(T))
+                put(f"prefill_attention_{label}", lambda: win(batch, T, T, kp, sc, **dict(kw)), flops=4.0 * H * hs * pairs)
+                cut = {nm: (t[:B] if nm == "gate" else t) for nm, t in kw.items()}
+                put(f"decode_attention_{label}", lambda: win(bd, B, 1, kp, sc, **dict(cut)), nbytes=2.0 * B * G * (W + kp) * hs * 2)
+            # norm over all heads + rotation in place, Nulezen's rotation alone, Lefalix's convolution + rotation + norm
+            am = vot.blocks[0].mixer
+            proj, fr = torch.randn(T, am.cols, device=dev, dtype=bf), am.freq(dev)
+            qv, kv_ = proj[:, : H * hs], proj[:, H * hs : (H + G) * hs]
+            turn = dict(freq=fr, rot_dims=hs // 2, interleaved=False)
+            put("norm_over_heads_rotation_votavik", lambda: K.head_rope(T, batch.row_pos, 1e-5, K.rope_seg(qv, qv, H, hs, norm_w=am.q_norm, norm_all=True, **turn),
+                                                                        K.rope_seg(kv_, kv_, G, hs, norm_w=am.k_norm, norm_all=True, **turn), dtype=bf, device=dev),
+                nbytes=T * (H + G) * hs * 4.0)
+            wm = lef.blocks[0].mixer.left
+            qkv, dst, tail, fl = torch.randn(T, wm.cols, device=dev, dtype=bf), torch.empty(T, wm.cols, device=dev, dtype=bf), torch.zeros(1, 3, wm.cols, device=dev, dtype=bf), wm.inv_freq(dev)
+            groups = [K.conv_group(wm.conv[: H * hs], dst[:, : H * hs], 0, H, hs, post=1, rot_dims=hs // 2, inv_freq=fl, rot_mscale=rot.magnitude, eps=1e-5),
+                      K.conv_group(wm.conv[H * hs : (H + G) * hs], dst[:, H * hs : (H + G) * hs], H * hs, G, hs, post=1, rot_dims=hs // 2, inv_freq=fl,
+                                   rot_mscale=rot.magnitude, eps=1e-5),
+                      K.conv_group(wm.conv[(H + G) * hs :], dst[:, (H + G) * hs :], (H + G) * hs, G, hs)]
+            put("short_conv_rotate_norm_lefalix", lambda: K.short_conv(qkv, groups, 4, tail, batch.seq_state, batch.row_seq), nbytes=T * wm.cols * 4.0)
+            # recurrences: q, k, v (and per-channel decays) in, o out; single rows read and write the states
+            Hl = H // 2
+            ql, kl, vl = (torch.randn(T, Hl * hs, device=dev, dtype=bf) for _ in range(3))
+            z, bias = torch.randn(T, Hl * hs, device=dev), torch.full((Hl * hs,), 3.0, device=dev, dtype=bf)
+            hd = vot.blocks[1].mixer.head_decay(dev)
+            st = torch.zeros(B, Hl * hs * hs, device=dev)
+            chan = dict(q_scale=hs ** -0.5, decay_bias=bias, tau=16.0)
+            rows_io = T * Hl * hs * (3 * 2 + 4.0)
+            put("prompt_linear_attention_per_channel_votavik", lambda: K.linear_attn(ql, kl, vl, st, batch.seq_state, T, Hl, hs, hs, decay_in=z, **chan),
+                nbytes=rows_io + T * Hl * hs * 4.0, us_per_token=0.0)
+            put("prompt_linear_attention_per_head_votavik", lambda: K.linear_attn(ql, kl, vl, st, batch.seq_state, T, Hl, hs, hs, silu=True, head_decay=hd),
+                nbytes=rows_io, us_per_token=0.0)
+            Gl = max(1, Hl // 2)
+            qf, kf = torch.nn.functional.normalize(torch.randn(T, Gl, hs, device=dev), dim=-1).view(T, -1), torch.nn.functional.normalize(torch.randn(T, Gl, hs, device=dev), dim=-1).view(T, -1)
+            vf, bt = torch.randn(T, Hl * hs, device=dev), torch.randn(T, Hl, device=dev, dtype=bf)
+            dc, dh = torch.randn(T, Hl * hs, device=dev, dtype=bf), torch.randn(T, Hl, device=dev, dtype=bf)
+            al, bc, bh = torch.zeros(Hl, device=dev, dtype=bf), torch.zeros(Hl * hs, device=dev, dtype=bf), torch.zeros(Hl, device=dev, dtype=bf)
+            std = torch.zeros(B, Hl * K.delta_rule_state_floats(hs, hs), device=dev)
+            drows = T * (2 * Gl + 2 * Hl) * hs * 4.0
+            put("prompt_delta_rule_per_channel_lefalix", lambda: K.delta_rule(qf, kf, vf, bt, dc, al, bc, std, batch.seq_state, Hl, Gl, hs, hs, True, max_rows=T),
+                nbytes=drows + T * Hl * hs * 2.0, us_per_token=0.0)
+            put("prompt_delta_rule_per_head_lefalix", lambda: K.delta_rule(qf, kf, vf, bt, dh, al, bh, std, batch.seq_state, Hl, Gl, hs, hs, False, max_rows=T),
+                nbytes=drows, us_per_token=0.0)
+            for key in [k_ for k_ in kern if "us_per_token" in kern[k_]]:
+                kern[key]["us_per_token"] = kern[key]["ms"] * 1e3 / T
+            states = 2.0 * B * Hl * hs * hs * 4
+            put("decode_linear_attention_per_channel_votavik", lambda: K.linear_attn(ql[:B], kl[:B], vl[:B], st, bd.seq_state, 1, Hl, hs, hs, decay_in=z[:B], **chan), nbytes=states)
+            put("decode_linear_attention_per_head_votavik", lambda: K.linear_attn(ql[:B], kl[:B], vl[:B], st, bd.seq_state, 1, Hl, hs, hs, silu=True, head_decay=hd), nbytes=states)
+            put("decode_delta_rule_per_channel_lefalix", lambda: K.delta_rule(qf[:B], kf[:B], vf[:B], bt[:B], dc[:B], al, bc, std, bd.seq_state, Hl, Gl, hs, hs, True, max_rows=1), nbytes=states)
+            put("decode_delta_rule_per_head_lefalix", lambda: K.delta_rule(qf[:B], kf[:B], vf[:B], bt[:B], dh[:B], al, bh, std, bd.seq_state, Hl, Gl, hs, hs, False, max_rows=1), nbytes=states)
+            # norm and gate behind the recurrence (fp32 in, gate in, out)
+            o, zg = torch.randn(T, Hl * hs, device=dev), torch.randn(T, Hl * hs, device=dev, dtype=bf)
+            w1, wa = torch.ones(hs, device=dev, dtype=bf), torch.ones(Hl * hs, device=dev, dtype=bf)
+            put("gated_norm_per_head_votavik_and_lefalix", lambda: K.gated_rms_heads(o, zg, w1, Hl, hs, K.GATE_SILU, 1e-5), nbytes=T * Hl * hs * 8.0)
+            put("gated_norm_all_heads_votavik", lambda: K.gated_rms_heads(o, zg, wa, 1, Hl * hs, K.GATE_SIGMOID, 1e-5), nbytes=T * Hl * hs * 8.0)
+            # residual kernels, feed-forwards, the per-layer token input
+            x, xs, act = torch.randn(T, d, device=dev, dtype=bf), torch.randn(T, d, device=dev), torch.empty(T, d, device=dev, dtype=bf)
+            vb, lb = vot.blocks[0], lef.blocks[1]
+            put("residual_layer_norm_votavik", lambda: K.sandwich_residual(xs, x, None, 1e-5, pre_w=vb.norm_2, pre_center=True, act=act), nbytes=T * d * 12.0)
+            put("residual_copy_votavik", lambda: K.sandwich_residual(xs, x, None, 1e-5, cast=act), nbytes=T * d * 12.0)
+            put("residual_normed_branch_layer_norm_votavik", lambda: K.sandwich_residual(xs, x, vb.side.norm, 1e-5, pre_w=vb.norm_1, pre_center=True, act=act), nbytes=T * d * 12.0)
+            put("residual_normed_branch_norm_lefalix", lambda: K.sandwich_residual(xs, x, lb.norm_1b, 1e-5, pre_w=lb.norm_2, act=act), nbytes=T * d * 12.0)
+            put("dense_mlp_clamped_votavik", lambda: vb.mlp(x), flops=6.0 * T * ff * d)
+            put("dense_mlp_gelu_lefalix", lambda: lb.mlp(x), flops=4.0 * T * dff * d)
+            toks = torch.randint(0, vocab, (T,), device=dev, dtype=torch.int32)
+            put("token_input_votavik", lambda: vb.side(x, toks, vot.side_embed), nbytes=T * (4.0 * d + 2.0 * 4 * side))
+            zz = torch.randn(T, side, device=dev, dtype=bf)
+            put("token_gate_votavik", lambda: K.token_gate(zz, toks, vot.side_embed, side, K.ACT_GELU_TANH), nbytes=T * side * 6.0)
+            put("gelu_lefalix_same_numbers", lambda: K.activation_(zz, K.ACT_GELU), nbytes=T * side * 4.0)
+            res["kernels"] = {k_: {a: (round(b_, 4) if isinstance(b_, float) else b_) for a, b_ in v_.items()} for k_, v_ in kern.items()}
+        out[name] = res
+        del vot, lef
+        torch.cuda.empty_cache()
+    print(json.dumps({"compare": "votavik", "layers": 4, "prompt": T, "context": T, "dtype": "bf16", "data": "synthetic, random weights",
+                      "l2": "flushed between timed calls", "peaks": {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"],
+                                                                       "source": peak_source},
+                      "gpu_launches": int(K.launch_count() - launches0), "sizes": out}), flush=True)
+
+
 def main() -> None:
     # stdout carries exactly one JSON line: NCCL's own banner / debug lines (when the box sets NCCL_DEBUG) go to stderr
     os.environ.setdefault("NCCL_DEBUG_FILE", "/dev/stderr")
@@ -1112,11 +1278,14 @@ def main() -> None:
     ap.add_argument("--workload", choices=sorted(WORKLOADS), default="llama2-7b-nf4-bs1")
     ap.add_argument("--layers", type=int, default=None, help="debug only: build fewer blocks (invalidates the number)")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--compare", choices=["pomipel", "lefalix", "fizadra", "nulezen"], default=None,
+    ap.add_argument("--compare", choices=["pomipel", "lefalix", "fizadra", "nulezen", "votavik"], default=None,
                     help="instead of the default workload: prefill / decode throughput of that design beside the closest existing model")
     ap.add_argument("--sizes", default=None, help=f"--compare: comma-separated subset of {sorted(ARCH_SIZES)} (the same names for both designs)")
     ap.add_argument("--prompt", type=int, default=2048, help="--compare: prompt and context length")
     args = ap.parse_args()
+    if args.compare == "votavik":
+        run_votavik_compare(args)
+        return
     if args.compare == "nulezen":
         run_nulezen_compare(args)
         return

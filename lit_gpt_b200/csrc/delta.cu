@@ -237,6 +237,42 @@ __global__ void __launch_bounds__(128) gated_rms_heads_kernel(const float* __res
   }
 }
 
+// the same for wide heads (all heads of a row normed together, say): one CTA per (row, head), eight numbers per access
+template <typename T>
+__global__ void __launch_bounds__(128) gated_rms_wide_kernel(const float* __restrict__ o, int64_t ldo, const T* __restrict__ z, int64_t ldz,
+                                                             const T* __restrict__ weight, T* __restrict__ out, int64_t ld_out, int dv, int gate, float eps) {
+  __shared__ float s_part[4];
+  griddep_launch();
+  griddep_wait();
+  const int64_t row = blockIdx.x, at = (int64_t)blockIdx.y * dv;
+  const float* orow = o + row * ldo + at;
+  const T* zrow = z + row * ldz + at;
+  T* yrow = out + row * ld_out + at;
+  float ss = 0.f;
+  for (int i = threadIdx.x * 8; i < dv; i += 1024) {
+    float v[8];
+    load8(orow + i, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss = fmaf(v[j], v[j], ss);
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0) s_part[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  const float rstd = 1.0f / sqrtf((s_part[0] + s_part[1] + s_part[2] + s_part[3]) / (float)dv + eps);
+  for (int i = threadIdx.x * 8; i < dv; i += 1024) {
+    float v[8], g[8], w[8];
+    load8(orow + i, v);
+    load8(zrow + i, g);
+    load8(weight + i, w);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const float sg = 1.0f / (1.0f + expf(-g[j]));
+      v[j] = v[j] * rstd * w[j] * (gate == 1 ? g[j] * sg : sg);
+    }
+    store8(yrow + i, v);
+  }
+}
+
 }  // namespace
 
 }  // namespace b200
@@ -286,6 +322,13 @@ int b200_gated_rms_heads(const float* o, int64_t ldo, const void* z, int64_t ldz
   B200_CHECK_ARG(o && z && weight && out, "b200_gated_rms_heads: null pointer");
   B200_CHECK_ARG(rows > 0 && rows <= 0x7fffffff && heads > 0 && (heads + 3) / 4 <= 65535 && dv > 0, "b200_gated_rms_heads: bad shape");
   B200_CHECK_ARG(gate == 1 || gate == 2, "b200_gated_rms_heads: gate is 1 (silu) or 2 (sigmoid)");
+  const size_t esz = dtype == B200_F32 ? 4 : 2;
+  auto al = [](const void* p, int64_t bytes) { return ((reinterpret_cast<uintptr_t>(p) | (uintptr_t)bytes) & 15) == 0; };
+  if (dv >= 256 && dv % 8 == 0 && heads <= 65535 && al(o, ldo * 4) && al(z, ldz * esz) && al(weight, 0) && al(out, ld_out * esz)) {
+    B200_FLOAT_TYPES(dtype, T, B200_CUDA(launch(gated_rms_wide_kernel<T>, dim3((unsigned)rows, (unsigned)heads), dim3(128), 0, (cudaStream_t)stream, o, ldo,
+                                                 (const T*)z, ldz, (const T*)weight, (T*)out, ld_out, dv, gate, eps)));
+    return B200_OK;
+  }
   B200_FLOAT_TYPES(dtype, T, B200_CUDA(launch(gated_rms_heads_kernel<T>, dim3((unsigned)rows, (unsigned)((heads + 3) / 4)), dim3(128), 0,
                                                (cudaStream_t)stream, o, ldo, (const T*)z, ldz, (const T*)weight, (T*)out, ld_out, heads, dv, gate, eps)));
   return B200_OK;

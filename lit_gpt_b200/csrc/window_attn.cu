@@ -252,6 +252,12 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
   const int lo = max(0, pos - A.window + 1);
   const int nk = min(A.keep, lo), n = nk + pos - lo + 1;           // visible: 0 .. nk - 1 (kept), then lo .. pos; entry j of n:
   auto position = [&](int j) { return j < nk ? j : lo + j - nk; };
+  // cache row of a visible position within the slot: the row's own ring place, and from there back by the distance (no division per key)
+  const int keep = A.keep, here = pos < keep ? 0 : (pos - keep) % A.ring;
+  auto ring_row = [&](int p) {
+    const int r = here - (pos - p);
+    return p < keep ? p : keep + (r < 0 ? r + A.ring : r);
+  };
   float* const qs = wd_smem;                        // [dk rounded up to 8]
   float* const sc = qs + ((dk + 7) & ~7);           // [window + keep rounded up to 4]
   float* const part = sc + ((A.window + A.keep + 3) & ~3);   // [value rows][dv]
@@ -260,8 +266,11 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
   const T* const vr = reinterpret_cast<const T*>(A.v_ring);
   const T* const k_now = reinterpret_cast<const T*>(A.k) + (int64_t)row * A.ldk + (int64_t)g * dk;
   const T* const v_now = reinterpret_cast<const T*>(A.v) + (int64_t)row * A.ldv + (int64_t)g * dv;
-  auto key_row = [&](int p) { return p == pos ? k_now : kr + wa_ring_row(slot, A.ring, A.keep, p) * G * dk + (int64_t)g * dk; };
-  auto value_row = [&](int p) { return p == pos ? v_now : vr + wa_ring_row(slot, A.ring, A.keep, p) * G * dv + (int64_t)g * dv; };
+  const int64_t rows0 = (int64_t)slot * (A.ring + keep);
+  const T* const k0 = kr + rows0 * G * dk + (int64_t)g * dk;
+  const T* const v0 = vr + rows0 * G * dv + (int64_t)g * dv;
+  auto key_row = [&](int p) { return p == pos ? k_now : k0 + (int64_t)ring_row(p) * (G * dk); };
+  auto value_row = [&](int p) { return p == pos ? v_now : v0 + (int64_t)ring_row(p) * (G * dv); };
   for (int d = tid; d < dk; d += kWdThreads) qs[d] = load_as_float(reinterpret_cast<const T*>(A.q), (int64_t)row * A.ldq + (int64_t)h * dk + d) * A.scale_log2;
   __syncthreads();
   float mx = -INFINITY;

@@ -150,3 +150,11 @@ def forward(cfg: dict, weights: Dict[str, torch.Tensor], tokens: List[int], retu
         seen.append(x.clone())
     logits = layer_norm(x, W["final.norm"], eps) @ W["head"].T
     return (logits, seen) if return_layers else logits
+
+
+def greedy(cfg: dict, weights: Dict[str, torch.Tensor], prompt: List[int], new_tokens: int) -> List[int]:
+    """prompt + greedily chosen continuation, recomputing everything for every token."""
+    seq = list(prompt)
+    for _ in range(new_tokens):
+        seq.append(int(forward(cfg, weights, seq)[-1].argmax()))
+    return seq

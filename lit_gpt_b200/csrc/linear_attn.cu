@@ -60,21 +60,32 @@ __device__ __forceinline__ float silu_f(float z) {
   return z / (1.0f + expf(-z));
 }
 
-// eight neighbouring elements of a row, zero beyond `n`
+// Eight neighbouring elements of a row as they lie in memory (zero beyond `n`): converted only when they are put into shared memory, so
+// that nothing waits for the loads of the next tile while the current one is walked.
 template <typename T>
-__device__ __forceinline__ void row8(const T* row, int i0, int n, bool vec, bool ok, float (&f)[8]) {
-  if (ok && vec && i0 + 8 <= n) {
-    load8(row + i0, f);
-  } else {
+struct alignas(16) Raw8 {
+  T e[8];
+  __device__ __forceinline__ void load(const T* row, int i0, int n, bool vec, bool ok) {
+    uint4* w = reinterpret_cast<uint4*>(e);
+    constexpr int W = sizeof(T) / 2;   // 16-byte words
 #pragma unroll
-    for (int j = 0; j < 8; ++j) f[j] = ok && i0 + j < n ? load_as_float(row, i0 + j) : 0.f;
+    for (int j = 0; j < W; ++j) w[j] = make_uint4(0, 0, 0, 0);
+    if (!ok) return;
+    if (vec && i0 + 8 <= n) {
+#pragma unroll
+      for (int j = 0; j < W; ++j) w[j] = reinterpret_cast<const uint4*>(row + i0)[j];
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) if (i0 + j < n) e[j] = row[i0 + j];
+    }
   }
-}
+  __device__ __forceinline__ void floats(float (&f)[8]) const { load8(e, f); }
+};
 
 // MODE 0: slot state -> slot state with read-out; 1: from zero, contribution and decay product to the workspace, no read-out;
 // 2: from the piece's starting state in the workspace, read-out only.
 template <typename T, int LK, int KPL, bool CHANNEL, int MODE>
-__global__ void __launch_bounds__(kLaThreads) walk_kernel(LaArgs A) {
+__global__ void __launch_bounds__(kLaThreads, sizeof(T) == 2 && KPL <= 8 ? 5 : 1) walk_kernel(LaArgs A) {
   constexpr int NC = kLaNC, DKP = LK * KPL, TT = kLaTile / DKP, GROUPS = kLaThreads / LK, COLS = GROUPS * NC;
   constexpr int NVV = (TT * COLS / 8 + kLaThreads - 1) / kLaThreads;   // 8-column pieces of a value tile per thread
   constexpr int K4 = KPL / 4;
@@ -136,58 +147,56 @@ __global__ void __launch_bounds__(kLaThreads) walk_kernel(LaArgs A) {
   const T* const qp = reinterpret_cast<const T*>(A.q) + (int64_t)h * dk;
   const T* const vp = reinterpret_cast<const T*>(A.v) + (int64_t)h * dv;
   const int st = tid / (DKP / 8), si = (tid % (DKP / 8)) * 8;          // this thread's token of a tile and its eight keys there
-  float rbias[CHANNEL ? 8 : 1];
-  if (CHANNEL) {
-#pragma unroll
-    for (int j = 0; j < 8; ++j)
-      rbias[j] = !A.z_ready && si + j < dk ? load_as_float(reinterpret_cast<const T*>(A.bias), (int64_t)h * dk + si + j) : 0.f;
-  }
-  float rk[8], rq[MODE == 1 ? 1 : 8], rz[CHANNEL ? 8 : 1], rv[NVV][8];
+  Raw8<T> rk, rq, rv[NVV];
+  Raw8<float> rz;
   auto load_tile = [&](int t0) {
     const int nt = min(TT, len - t0);
     const int64_t row = first + t0 + st;
-    row8(kp + row * A.ldk, si, dk, A.vec_k, st < nt, rk);
-    if constexpr (MODE != 1) row8(qp + row * A.ldq, si, dk, A.vec_k, st < nt, rq);
-    if constexpr (CHANNEL) row8(A.z + row * A.ldz + (int64_t)h * dk, si, dk, A.vec_z, st < nt, rz);
+    rk.load(kp + row * A.ldk, si, dk, A.vec_k, st < nt);
+    if constexpr (MODE != 1) rq.load(qp + row * A.ldq, si, dk, A.vec_k, st < nt);
+    if constexpr (CHANNEL) rz.load(A.z + row * A.ldz + (int64_t)h * dk, si, dk, A.vec_z, st < nt);
 #pragma unroll
     for (int n = 0; n < NVV; ++n) {
       const int idx = tid + n * kLaThreads, t = idx / (COLS / 8), c = (idx % (COLS / 8)) * 8;
-      row8(vp + (int64_t)(first + t0 + t) * A.ldv, col0 + c, dv, A.vec_v, t < nt && col0 + c < dv, rv[n]);
+      rv[n].load(vp + (int64_t)(first + t0 + t) * A.ldv, col0 + c, dv, A.vec_v, t < nt && col0 + c < dv);
     }
   };
   auto store_tile = [&](int nt) {
-    if (st < nt) {
+    float f[8];
+    auto activate = [&]() {
       if (A.act) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) rk[j] = silu_f<T>(rk[j]);
+        for (int j = 0; j < 8; ++j) f[j] = silu_f<T>(f[j]);
       }
-      store8(ks + st * DKP + si, rk);
+    };
+    if (st < nt) {
+      rk.floats(f);
+      activate();
+      store8(ks + st * DKP + si, f);
       if constexpr (MODE != 1) {
-        if (A.act) {
+        rq.floats(f);
+        activate();
 #pragma unroll
-          for (int j = 0; j < 8; ++j) rq[j] = silu_f<T>(rq[j]);
-        }
-#pragma unroll
-        for (int j = 0; j < 8; ++j) rq[j] *= A.q_scale;
-        store8(qs + st * DKP + si, rq);
+        for (int j = 0; j < 8; ++j) f[j] *= A.q_scale;
+        store8(qs + st * DKP + si, f);
       }
       if constexpr (CHANNEL) {
+        rz.floats(f);
         if (!A.z_ready) {
+          const T* bias = reinterpret_cast<const T*>(A.bias) + (int64_t)h * dk;
 #pragma unroll
-          for (int j = 0; j < 8; ++j) rz[j] = channel_decay(rz[j] + rbias[j], A.inv_tau);
+          for (int j = 0; j < 8; ++j) f[j] = channel_decay(f[j] + (si + j < dk ? load_as_float(bias, si + j) : 0.f), A.inv_tau);
         }
-        store8(gs + st * DKP + si, rz);
+        store8(gs + st * DKP + si, f);
       }
     }
 #pragma unroll
     for (int n = 0; n < NVV; ++n) {
       const int idx = tid + n * kLaThreads, t = idx / (COLS / 8), c = (idx % (COLS / 8)) * 8;
       if (t < nt) {
-        if (A.act) {
-#pragma unroll
-          for (int j = 0; j < 8; ++j) rv[n][j] = silu_f<T>(rv[n][j]);
-        }
-        store8(vs + t * COLS + c, rv[n]);
+        rv[n].floats(f);
+        activate();
+        store8(vs + t * COLS + c, f);
       }
     }
   };

@@ -4,7 +4,7 @@ the replay of a recorded trace of steps.
 ``Session`` owns what a set of live requests needs: the model's caches (grown when more requests are live than there are
 slots), one cache slot and the number of cached tokens per request.  ``Session.step`` is the one step function: every entry
 brings the next tokens of a request, all entries run as one ragged batch (the model's ``step``), finished requests give their
-slots back; the model is any that serves sequences from slots (``ragged.SlotServed`` with a ``step``: Pomipel, Lefalix).  ``generate_batch`` schedules prompts through it (prefill together, then one token per live request and step,
+slots back; the model is any that serves sequences from slots (``ragged.SlotServed`` with a ``step``).  ``generate_batch`` schedules prompts through it (prefill together, then one token per live request and step,
 shorter requests leaving the batch early); ``Replayer`` feeds it recorded steps instead of sampled tokens.
 """
 from __future__ import annotations

@@ -445,10 +445,15 @@ int b200_latent_decode_tune(int force_any_size_kernel);
  * the `keep` best of `n_group` equal groups of neighbours (group rank = sum of its two largest corrected scores, or the largest
  * with B200_ROUTE_GROUP_MAX); weights[t, k] = s of the chosen expert, not renormalised.  B200_ROUTE_TOPK_SOFTMAX: s is the raw logit,
  * the largest logits are chosen and the weights are a softmax among those `top` logits.  B200_ROUTE_BIAS: `correction` is a bias
- * added to the logit itself (it enters the scores) instead of a selection-only term. */
+ * added to the logit itself (it enters the scores) instead of a selection-only term.  gate_w (d numbers, with gate; NULL: none): also
+ * gate[t] = sigmoid(gate_w . x), the gate of a shared expert. */
 enum b200_route_flags { B200_ROUTE_SOFTMAX = 1, B200_ROUTE_GROUP_MAX = 2, B200_ROUTE_TOPK_SOFTMAX = 4, B200_ROUTE_BIAS = 8 };
 int b200_moe_route(const void* x, const void* w_router, const void* correction, int32_t* ids, float* weights, int64_t tokens, int d,
-                   int n_expert, int top, int n_group, int keep, int flags, int dtype, b200_stream_t stream);
+                   int n_expert, int top, int n_group, int keep, int flags, const void* gate_w, float* gate, int dtype, b200_stream_t stream);
+/* the same choice for B200_ROUTE_TOPK_SOFTMAX from logits (tokens, ld) fp32 that a matrix product left: the largest `top` <= 32 of the first
+ * n_expert columns; with gate, gate[t] = sigmoid(column n_expert) */
+int b200_moe_route_logits(const float* logits, int64_t ld, int32_t* ids, float* weights, float* gate, int64_t tokens, int n_expert, int top,
+                          b200_stream_t stream);
 /* counting sort of the (token, choice) pairs by expert: expert_off[E + 1], tile_off[E + 1] (64-row tiles), slot_token[tokens * top],
  * slot_of[tokens * top] */
 int b200_moe_plan(const int32_t* ids, int64_t tokens, int top, int n_expert, int32_t* expert_off, int32_t* tile_off, int32_t* slot_token,
@@ -458,9 +463,12 @@ int b200_moe_gemm(const void* a, int64_t lda, const int32_t* row_src, const void
                   const int32_t* tile_off, int64_t rows, int n_expert, int n, int k, int sqrelu, int dtype, b200_stream_t stream);
 /* few tokens: hidden = relu(W_up[e] x)^2 per (token, choice) -- gated 1: silu(W_up[e][:ff] x) * (W_up[e][ff:] x) with 2 ff rows per
  * expert; gated 2: g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit) --,
- * out[t] = sum_k weights[t, k] * W_down[e_k] hidden[t, k] */
+ * out[t] = sum_k weights[t, k] * W_down[e_k] hidden[t, k].  With gated 1 also a shared expert of the same form that every token uses
+ * (shared_up (2 shared_ff, d), shared_down (d, shared_ff); NULL: none): its result goes to shared_out (tokens, d) by way of shared_hidden
+ * (tokens, shared_ff). */
 int b200_moe_gemv(const void* x, const int32_t* ids, const float* weights, const void* w_up, const void* w_down, void* hidden, void* out,
-                  int64_t tokens, int top, int d, int ff, int gated, float limit, float alpha, int dtype, b200_stream_t stream);
+                  int64_t tokens, int top, int d, int ff, int gated, float limit, float alpha, const void* shared_up, const void* shared_down,
+                  int shared_ff, void* shared_hidden, void* shared_out, int dtype, b200_stream_t stream);
 int b200_moe_combine(const void* y, const int32_t* slot_of, const float* weights, void* out, int64_t tokens, int top, int d, int dtype,
                      b200_stream_t stream);
 
@@ -514,6 +522,17 @@ typedef struct b200_scaled_residual_args {
   int d, dtype;
 } b200_scaled_residual_args;
 int b200_scaled_residual(const b200_scaled_residual_args* args, b200_stream_t stream);
+/* x += mult * scale * (y + gate[row] * y1) (fp32 stream, in place; y1, gate (fp32, one per row) and scale (d numbers) optional) with
+ * y = y0[row], or sum_k wts[row, k] * y0[slot_of[row, k]] over `top` rows; act = dtype(x / sqrt(mean(x^2) + eps) * w), or * (1 + w) with
+ * plus_one (w NULL: skipped).  y0, y1, scale, w and act are `dtype`. */
+typedef struct b200_gated_residual_args {
+  const void* y0; const int32_t* slot_of; const float* wts; int top;
+  const void* y1; const float* gate; const void* scale; float mult;
+  float* x; const void* w; int plus_one; void* act;
+  int64_t rows;
+  int d; float eps; int dtype;
+} b200_gated_residual_args;
+int b200_gated_residual(const b200_gated_residual_args* args, b200_stream_t stream);
 
 /* One group of heads of a short causal convolution (see b200_short_conv). */
 typedef struct b200_conv_group {
@@ -558,9 +577,9 @@ typedef struct b200_delta_rule_args {
 } b200_delta_rule_args;
 int64_t b200_delta_rule_state_floats(int dk, int dv);
 int b200_delta_rule(const b200_delta_rule_args* args, b200_stream_t stream);
-/* out[row, h, :] = dtype(o / sqrt(mean(o^2) + eps) * weight * gate(z)) per head; gate 1 silu, 2 sigmoid */
+/* out[row, h, :] = dtype(o / sqrt(mean(o^2) + eps) * weight * gate(z) * out_scale) per head; gate 1 silu, 2 sigmoid; weight NULL: none */
 int b200_gated_rms_heads(const float* o, int64_t ldo, const void* z, int64_t ldz, const void* weight, void* out, int64_t ld_out, int64_t rows,
-                         int heads, int dv, int gate, float eps, int dtype, b200_stream_t stream);
+                         int heads, int dv, int gate, float eps, float out_scale, int dtype, b200_stream_t stream);
 
 /* Sliding-window attention with a per-head sink logit in the softmax denominator (sink NULL: none).  Row at position i sees
  * positions i - window < j <= i: those of this step from k / v (rows, n_kv_head * dk | dv), older ones from the rings
@@ -583,10 +602,11 @@ typedef struct b200_window_attn_args {
   /* optional (0: none): positions j < keep stay visible whatever the window; score <- softcap * tanh(score / softcap) after the scale.
    * The rings then hold keep + ring rows per slot: position p in row p when p < keep, else in row keep + (p - keep) % ring. */
   int keep; float softcap;
+  float out_scale;   /* the output is multiplied by this */
 } b200_window_attn_args;
 int b200_window_attn(const b200_window_attn_args* args, b200_stream_t stream);
 /* The tensor-core tiles of b200_attn_prefill_window for the same description, without distance bias and without touching the rings:
- * bf16, dk and dv multiples of 8 up to 128 (they may differ), every sequence at position 0, leading dimensions of q, k, v multiples of 8
+ * bf16, dk a multiple of 8 up to 128, dv one up to 256, every sequence at position 0, leading dimensions of q, k, v multiples of 8
  * elements, q / k / v / seqs 16-byte aligned. */
 int b200_window_attn_tiles(const b200_window_attn_args* args, b200_stream_t stream);
 /* test knob: non-zero keeps single-row steps on the tiled kernel; returns the previous setting */
@@ -604,7 +624,8 @@ int b200_ring_store_keep(const void* k, int64_t ldk, const void* v, int64_t ldv,
  * o = S^T q.  q, k (rows, heads * dk) and v (rows, heads * dv) are projections in `dtype`, each through silu when act is 1, q then times
  * q_scale.  Decays: head_decay[heads], fixed -- or decay_in (rows, heads * dk) fp32 raw with decay_bias (heads * dk, `dtype`) and tau,
  * g = sigmoid(decay_in + decay_bias)^(1 / tau) (decay_in is scratch: its rows may be overwritten).  A sequence at position 0 starts from
- * S = 0.  Long prompts run in pieces side by side, for which the workspace holds a state per piece. */
+ * S = 0.  Long prompts run in pieces side by side, for which the workspace holds a state per piece.  qk_f32 (with head_decay only): q and k
+ * are fp32 whatever `dtype` is. */
 typedef struct b200_linear_attn_args {
   const void* q; const void* k; const void* v;
   int64_t ldq, ldk, ldv;
@@ -617,6 +638,7 @@ typedef struct b200_linear_attn_args {
   int64_t rows; int max_rows;       /* rows of the step; of its longest sequence */
   int heads, dk, dv, dtype;
   void* workspace; size_t workspace_bytes;
+  int qk_f32;
 } b200_linear_attn_args;
 size_t b200_linear_attn_workspace_bytes(int64_t rows, int max_rows, int n_seqs, int heads, int dk, int dv);
 int b200_linear_attn(const b200_linear_attn_args* args, b200_stream_t stream);
@@ -640,13 +662,14 @@ int b200_depth_residual(const b200_depth_residual_args* args, b200_stream_t stre
  * out + out_rows[row] * ld_out + h * out_stride (out_rows NULL: the row itself; a row < 0 is skipped; in place allowed).  norm_w
  * (dim numbers, NULL: no norm) is the weight of an RMS norm over the head; dimensions [rot_off, rot_off + rot_dims) turn by
  * position * freq[i] (fp32, or fp64 with freq_f64), pair i = (2 i, 2 i + 1) when interleaved, else (i, i + rot_dims / 2), cos and sin
- * times mag.  norm_all: one norm over all heads of the row at once (in_stride = dim), norm_w then holds heads * dim numbers. */
+ * times mag.  norm_all: one norm over all heads of the row at once (in_stride = dim), norm_w then holds heads * dim numbers.  out_f32: `out` is
+ * fp32 whatever the dtype is (not in place then).  One to four groups per call. */
 typedef struct b200_head_rope_seg {
   const void* in; void* out; const void* norm_w; const void* freq; const int64_t* out_rows;
   int64_t ld_in, ld_out;
   int heads, dim, in_stride, out_stride, rot_off, rot_dims, interleaved;
   float mag;
-  int norm_all, freq_f64;
+  int norm_all, freq_f64, out_f32;
 } b200_head_rope_seg;
 int b200_head_rope(const b200_head_rope_seg* segs, int n_segs, const int32_t* row_pos, int64_t rows, float eps, int dtype, b200_stream_t stream);
 /* Causal attention over cached keys and values in which the heads' scores are mixed before the softmax:

@@ -104,7 +104,7 @@ class DepthResidualArgs(ctypes.Structure):  # mirrors b200_depth_residual_args
 class HeadRopeSeg(ctypes.Structure):  # mirrors b200_head_rope_seg
     _fields_ = [("inp", c_void_p), ("out", c_void_p), ("norm_w", c_void_p), ("freq", c_void_p), ("out_rows", c_void_p), ("ld_in", c_int64),
                 ("ld_out", c_int64), ("heads", c_int), ("dim", c_int), ("in_stride", c_int), ("out_stride", c_int), ("rot_off", c_int),
-                ("rot_dims", c_int), ("interleaved", c_int), ("mag", c_float), ("norm_all", c_int), ("freq_f64", c_int)]
+                ("rot_dims", c_int), ("interleaved", c_int), ("mag", c_float), ("norm_all", c_int), ("freq_f64", c_int), ("out_f32", c_int)]
 
 
 class TalkAttnArgs(ctypes.Structure):  # mirrors b200_talk_attn_args
@@ -139,7 +139,8 @@ class WindowAttnArgs(ctypes.Structure):  # mirrors b200_window_attn_args
                 ("ldo", c_int64), ("k_ring", c_void_p), ("v_ring", c_void_p), ("sink", c_void_p), ("seqs", c_void_p), ("n_seqs", c_int),
                 ("max_q_len", c_int), ("ring", c_int), ("n_head", c_int), ("n_kv_head", c_int), ("dk", c_int), ("dv", c_int), ("window", c_int),
                 ("scale", c_float), ("dtype", c_int), ("row_seq", c_void_p), ("rows", c_int64), ("dist_r1", c_void_p), ("dist_r2", c_void_p),
-                ("gate", c_void_p), ("ldg", c_int64), ("gate_mode", c_int), ("keep", c_int), ("softcap", c_float)]
+                ("gate", c_void_p), ("ldg", c_int64), ("gate_mode", c_int), ("keep", c_int), ("softcap", c_float),
+                ("out_scale", c_float)]
 
 
 class LinearAttnArgs(ctypes.Structure):  # mirrors b200_linear_attn_args
@@ -147,7 +148,13 @@ class LinearAttnArgs(ctypes.Structure):  # mirrors b200_linear_attn_args
                 ("q_scale", c_float), ("decay_in", c_void_p), ("ld_decay", c_int64), ("decay_bias", c_void_p), ("tau", c_float), ("head_decay", c_void_p),
                 ("state", c_void_p), ("state_slot_stride", c_int64), ("out", c_void_p), ("ldo", c_int64), ("seqs", c_void_p), ("n_seqs", c_int),
                 ("rows", c_int64), ("max_rows", c_int), ("heads", c_int), ("dk", c_int), ("dv", c_int), ("dtype", c_int), ("workspace", c_void_p),
-                ("workspace_bytes", c_size_t)]
+                ("workspace_bytes", c_size_t), ("qk_f32", c_int)]
+
+
+class GatedResidualArgs(ctypes.Structure):  # mirrors b200_gated_residual_args
+    _fields_ = [("y0", c_void_p), ("slot_of", c_void_p), ("wts", c_void_p), ("top", c_int), ("y1", c_void_p), ("gate", c_void_p), ("scale", c_void_p),
+                ("mult", c_float), ("x", c_void_p), ("w", c_void_p), ("plus_one", c_int), ("act", c_void_p), ("rows", c_int64), ("d", c_int), ("eps", c_float),
+                ("dtype", c_int)]
 
 
 class ScaledResidualArgs(ctypes.Structure):  # mirrors b200_scaled_residual_args
@@ -178,12 +185,14 @@ _CORE_SIGNATURES = {
     "b200_latent_decode_workspace_bytes": (c_size_t, [c_int, c_int, c_int, c_int]),
     "b200_latent_decode": (c_int, [ctypes.POINTER(LatentDecodeArgs), c_void_p]),
     "b200_latent_decode_tune": (c_int, [c_int]),
-    "b200_moe_route": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "b200_moe_route": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p,
+                               c_int, c_void_p]),
+    "b200_moe_route_logits": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_void_p]),
     "b200_moe_plan": (c_int, [c_void_p, c_int64, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
     "b200_moe_gemm": (c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_int,
                               c_void_p]),
     "b200_moe_gemv": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_int, c_float, c_float,
-                              c_int, c_void_p]),
+                              c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p]),
     "b200_moe_combine": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p]),
     "b200_sandwich_residual": (c_int, [ctypes.POINTER(SandwichArgs), c_void_p]),
     "b200_activation": (c_int, [c_void_p, c_int64, c_int, c_int, c_void_p]),
@@ -191,13 +200,14 @@ _CORE_SIGNATURES = {
     "b200_xielu": (c_int, [c_void_p, c_int64, c_void_p, c_int, c_void_p]),
     "b200_glu_clamped": (c_int, [c_void_p, c_void_p, c_int64, c_int, c_float, c_float, c_int, c_void_p]),
     "b200_scaled_residual": (c_int, [ctypes.POINTER(ScaledResidualArgs), c_void_p]),
+    "b200_gated_residual": (c_int, [ctypes.POINTER(GatedResidualArgs), c_void_p]),
     "b200_short_conv": (c_int, [c_void_p, c_int64, ctypes.POINTER(ConvGroup), c_int, c_int, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_int64, c_int,
                                 c_void_p]),
     "b200_conv_tail_update": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_int, c_int, c_void_p, c_int, c_int, c_void_p]),
     "b200_delta_rule_state_floats": (c_int64, [c_int, c_int]),
     "b200_delta_rule": (c_int, [ctypes.POINTER(DeltaRuleArgs), c_void_p]),
-    "b200_gated_rms_heads": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int64, c_int, c_int, c_int, c_float, c_int,
-                                     c_void_p]),
+    "b200_gated_rms_heads": (c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int64, c_int, c_int, c_int, c_float, c_float,
+                                     c_int, c_void_p]),
     "b200_window_attn": (c_int, [ctypes.POINTER(WindowAttnArgs), c_void_p]),
     "b200_window_attn_tune": (c_int, [c_int]),
     "b200_window_attn_tiles": (c_int, [ctypes.POINTER(WindowAttnArgs), c_void_p]),

@@ -64,6 +64,7 @@ struct PfView {
   // cap * log2(e), cap_in = 2 * scale / cap * log2(e) (0: no cap).
   int dk, dv, keep;
   float cap_log2, cap_in;
+  float out_scale;   // the output is multiplied by this
 };
 
 constexpr int kPfBiasTabMax = 8192;   // distances a CTA tabulates at most (32 KB)
@@ -364,6 +365,7 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     iA = cA / (lA * cA + exp2f(sk - eA));
     iB = cB / (lB * cB + exp2f(sk - eB));
   }
+  if constexpr (EX) { iA *= vw.out_scale; iB *= vw.out_scale; }
   const int gmode = vw.seqs && vw.gate ? vw.gate_mode : 0;
   const int dv = EX ? vw.dv : HV;
   // the gate's sigmoid with the fast exponential and reciprocal: the product is rounded to bf16 right after
@@ -587,8 +589,8 @@ extern "C" int b200_attn_prefill_window_ex(const void* q, int64_t ldq, const voi
   return B200_OK;
 }
 
-// The same tiles with kept first positions, a soft cap, and query / key and value sizes of their own (multiples of 8 up to 128, padded
-// with zeros to 64 or 128 in shared memory), described as b200_window_attn describes them; the sequences start in this step.
+// The same tiles with kept first positions, a soft cap, and query / key and value sizes of their own (multiples of 8 up to 128 and
+// 256, padded with zeros to a multiple of 64 in shared memory), described as b200_window_attn describes them; the sequences start in this step.
 extern "C" int b200_window_attn_tiles(const b200_window_attn_args* a, b200_stream_t stream) {
   B200_CHECK_ARG(a && a->q && a->k && a->v && a->out && a->seqs, "b200_window_attn_tiles: null pointer");
   B200_CHECK_ARG(!a->dist_r1 && !a->dist_r2, "b200_window_attn_tiles: no distance bias here");
@@ -596,8 +598,8 @@ extern "C" int b200_window_attn_tiles(const b200_window_attn_args* a, b200_strea
   B200_CHECK_ARG(a->n_seqs > 0 && a->n_seqs <= 65535 && a->max_q_len > 0 && a->n_head > 0 && a->n_head <= 65535 && a->n_kv_head > 0 &&
                      a->n_head % a->n_kv_head == 0 && a->window > 0 && a->keep >= 0 && a->softcap >= 0.f && a->scale > 0.f,
                  "b200_window_attn_tiles: bad shape");
-  B200_CHECK_ARG(a->dtype == B200_BF16 && a->dk > 0 && a->dk <= 128 && a->dk % 8 == 0 && a->dv > 0 && a->dv <= 128 && a->dv % 8 == 0,
-                 "b200_window_attn_tiles: bf16 heads of multiples of 8 numbers, at most 128");
+  B200_CHECK_ARG(a->dtype == B200_BF16 && a->dk > 0 && a->dk <= 128 && a->dk % 8 == 0 && a->dv > 0 && a->dv <= 256 && a->dv % 8 == 0,
+                 "b200_window_attn_tiles: bf16 heads of multiples of 8 numbers, at most 128 (keys) and 256 (values)");
   B200_CHECK_ARG(((a->ldq | a->ldk | a->ldv) & 7) == 0 && (a->ldo & 1) == 0, "b200_window_attn_tiles: leading dimensions must be multiples of 8 elements");
   B200_CHECK_ARG(((reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->k) | reinterpret_cast<uintptr_t>(a->v) |
                    reinterpret_cast<uintptr_t>(a->seqs)) & 15) == 0 && (reinterpret_cast<uintptr_t>(a->out) & 3) == 0,
@@ -606,13 +608,20 @@ extern "C" int b200_window_attn_tiles(const b200_window_attn_args* a, b200_strea
   const PfView vw{0, a->dk, a->ldq, 0, a->dk, a->ldk, 0, a->dv, a->ldv, 0, a->ldo, reinterpret_cast<const int4*>(a->seqs), a->window,
                   reinterpret_cast<const __nv_bfloat16*>(a->sink), 1, nullptr, 0, a->gate_mode ? reinterpret_cast<const __nv_bfloat16*>(a->gate) : nullptr,
                   a->ldg, a->gate_mode, nullptr, 0, 0, 0, 0, nullptr, nullptr, 0, a->dk, a->dv, a->keep, a->softcap * kLog2e,
-                  a->softcap > 0.f ? 2.0f * a->scale / a->softcap * kLog2e : 0.f};
+                  a->softcap > 0.f ? 2.0f * a->scale / a->softcap * kLog2e : 0.f, a->out_scale};
   cudaStream_t st = (cudaStream_t)stream;
   const int H = a->n_head, G = a->n_kv_head;
-  if (a->dk > 64 && a->dv > 64) B200_CUDA((launch_prefill<128, int32_t, 0, 0, 128, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
-  else if (a->dk > 64) B200_CUDA((launch_prefill<128, int32_t, 0, 0, 64, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
-  else if (a->dv > 64) B200_CUDA((launch_prefill<64, int32_t, 0, 0, 128, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
-  else B200_CUDA((launch_prefill<64, int32_t, 0, 0, 64, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+  if (a->dk > 64) {
+    if (a->dv <= 64) B200_CUDA((launch_prefill<128, int32_t, 0, 0, 64, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+    else if (a->dv <= 128) B200_CUDA((launch_prefill<128, int32_t, 0, 0, 128, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+    else if (a->dv <= 192) B200_CUDA((launch_prefill<128, int32_t, 0, 0, 192, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+    else B200_CUDA((launch_prefill<128, int32_t, 0, 0, 256, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+  } else {
+    if (a->dv <= 64) B200_CUDA((launch_prefill<64, int32_t, 0, 0, 64, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+    else if (a->dv <= 128) B200_CUDA((launch_prefill<64, int32_t, 0, 0, 128, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+    else if (a->dv <= 192) B200_CUDA((launch_prefill<64, int32_t, 0, 0, 192, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+    else B200_CUDA((launch_prefill<64, int32_t, 0, 0, 256, true>(a->q, a->k, a->v, nullptr, a->out, a->n_seqs, a->max_q_len, H, G, 0, a->scale, st, &vw)));
+  }
   return B200_OK;
 }
 

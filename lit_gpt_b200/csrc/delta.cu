@@ -219,7 +219,7 @@ cudaError_t delta_launch(const DrArgs& A, bool channel, int n_seqs, cudaStream_t
 template <typename T>
 __global__ void __launch_bounds__(128) gated_rms_heads_kernel(const float* __restrict__ o, int64_t ldo, const T* __restrict__ z, int64_t ldz,
                                                               const T* __restrict__ weight, T* __restrict__ out, int64_t ld_out, int heads,
-                                                              int dv, int gate, float eps) {
+                                                              int dv, int gate, float eps, float out_scale) {
   griddep_launch();
   griddep_wait();
   const int lane = threadIdx.x & 31;
@@ -233,14 +233,15 @@ __global__ void __launch_bounds__(128) gated_rms_heads_kernel(const float* __res
   for (int i = lane; i < dv; i += 32) {
     const float zz = load_as_float(z, row * ldz + (int64_t)h * dv + i);
     const float sg = 1.0f / (1.0f + expf(-zz));
-    store_from_float(out, row * ld_out + (int64_t)h * dv + i, orow[i] * rstd * load_as_float(weight, i) * (gate == 1 ? zz * sg : sg));
+    store_from_float(out, row * ld_out + (int64_t)h * dv + i, orow[i] * rstd * (weight ? load_as_float(weight, i) : 1.0f) * (gate == 1 ? zz * sg : sg) * out_scale);
   }
 }
 
 // the same for wide heads (all heads of a row normed together, say): one CTA per (row, head), eight numbers per access
 template <typename T>
 __global__ void __launch_bounds__(128) gated_rms_wide_kernel(const float* __restrict__ o, int64_t ldo, const T* __restrict__ z, int64_t ldz,
-                                                             const T* __restrict__ weight, T* __restrict__ out, int64_t ld_out, int dv, int gate, float eps) {
+                                                             const T* __restrict__ weight, T* __restrict__ out, int64_t ld_out, int dv, int gate, float eps,
+                                                             float out_scale) {
   __shared__ float s_part[4];
   griddep_launch();
   griddep_wait();
@@ -263,11 +264,11 @@ __global__ void __launch_bounds__(128) gated_rms_wide_kernel(const float* __rest
     float v[8], g[8], w[8];
     load8(orow + i, v);
     load8(zrow + i, g);
-    load8(weight + i, w);
+    if (weight) load8(weight + i, w);
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
       const float sg = 1.0f / (1.0f + expf(-g[j]));
-      v[j] = v[j] * rstd * w[j] * (gate == 1 ? g[j] * sg : sg);
+      v[j] = v[j] * rstd * (weight ? w[j] : 1.0f) * (gate == 1 ? g[j] * sg : sg) * out_scale;
     }
     store8(yrow + i, v);
   }
@@ -318,19 +319,19 @@ int b200_delta_rule(const b200_delta_rule_args* a, b200_stream_t stream) {
 }
 
 int b200_gated_rms_heads(const float* o, int64_t ldo, const void* z, int64_t ldz, const void* weight, void* out, int64_t ld_out, int64_t rows,
-                         int heads, int dv, int gate, float eps, int dtype, b200_stream_t stream) {
-  B200_CHECK_ARG(o && z && weight && out, "b200_gated_rms_heads: null pointer");
+                         int heads, int dv, int gate, float eps, float out_scale, int dtype, b200_stream_t stream) {
+  B200_CHECK_ARG(o && z && out, "b200_gated_rms_heads: null pointer");
   B200_CHECK_ARG(rows > 0 && rows <= 0x7fffffff && heads > 0 && (heads + 3) / 4 <= 65535 && dv > 0, "b200_gated_rms_heads: bad shape");
   B200_CHECK_ARG(gate == 1 || gate == 2, "b200_gated_rms_heads: gate is 1 (silu) or 2 (sigmoid)");
   const size_t esz = dtype == B200_F32 ? 4 : 2;
   auto al = [](const void* p, int64_t bytes) { return ((reinterpret_cast<uintptr_t>(p) | (uintptr_t)bytes) & 15) == 0; };
   if (dv >= 256 && dv % 8 == 0 && heads <= 65535 && al(o, ldo * 4) && al(z, ldz * esz) && al(weight, 0) && al(out, ld_out * esz)) {
     B200_FLOAT_TYPES(dtype, T, B200_CUDA(launch(gated_rms_wide_kernel<T>, dim3((unsigned)rows, (unsigned)heads), dim3(128), 0, (cudaStream_t)stream, o, ldo,
-                                                 (const T*)z, ldz, (const T*)weight, (T*)out, ld_out, dv, gate, eps)));
+                                                 (const T*)z, ldz, (const T*)weight, (T*)out, ld_out, dv, gate, eps, out_scale)));
     return B200_OK;
   }
   B200_FLOAT_TYPES(dtype, T, B200_CUDA(launch(gated_rms_heads_kernel<T>, dim3((unsigned)rows, (unsigned)((heads + 3) / 4)), dim3(128), 0,
-                                               (cudaStream_t)stream, o, ldo, (const T*)z, ldz, (const T*)weight, (T*)out, ld_out, heads, dv, gate, eps)));
+                                               (cudaStream_t)stream, o, ldo, (const T*)z, ldz, (const T*)weight, (T*)out, ld_out, heads, dv, gate, eps, out_scale)));
   return B200_OK;
 }
 

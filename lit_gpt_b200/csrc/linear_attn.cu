@@ -2,7 +2,8 @@
 //
 //   per token:  S <- diag(g) S + k v^T      (g: one fixed decay per head, or one per head and key channel from the token)
 //               o  = S^T q                  (the read-out sees the token's own write)
-//   q, k, v come straight from the projections (bf16 or fp32), optionally through silu, q times a constant; with per-channel
+//   q, k, v come straight from the projections (bf16 or fp32), optionally through silu, q times a constant -- or q and k in fp32 from a
+//   step of their own (a rotation) beside values in the projections' dtype; with per-channel
 //   decays g = sigmoid(z + bias)^(1 / tau), all of it in fp32.
 //
 // walk_kernel goes through the tokens of one piece of a sequence in order.  The columns of S never mix: column j evolves from
@@ -84,8 +85,9 @@ struct alignas(16) Raw8 {
 
 // MODE 0: slot state -> slot state with read-out; 1: from zero, contribution and decay product to the workspace, no read-out;
 // 2: from the piece's starting state in the workspace, read-out only.
-template <typename T, int LK, int KPL, bool CHANNEL, int MODE>
-__global__ void __launch_bounds__(kLaThreads, sizeof(T) == 2 && KPL <= 8 ? 5 : 1) walk_kernel(LaArgs A) {
+// T: dtype of the values (and of the per-channel decays' bias), TQ: of queries and keys.
+template <typename T, typename TQ, int LK, int KPL, bool CHANNEL, int MODE>
+__global__ void __launch_bounds__(kLaThreads, sizeof(TQ) == 2 && KPL <= 8 ? 5 : (sizeof(T) == 2 && KPL <= 8 ? 4 : 1)) walk_kernel(LaArgs A) {
   constexpr int NC = kLaNC, DKP = LK * KPL, TT = kLaTile / DKP, GROUPS = kLaThreads / LK, COLS = GROUPS * NC;
   constexpr int NVV = (TT * COLS / 8 + kLaThreads - 1) / kLaThreads;   // 8-column pieces of a value tile per thread
   constexpr int K4 = KPL / 4;
@@ -143,11 +145,12 @@ __global__ void __launch_bounds__(kLaThreads, sizeof(T) == 2 && KPL <= 8 ? 5 : 1
   const float hd = CHANNEL ? 0.f : A.head_decay[h];
   const f2 hd2 = pk2(hd, hd);
 
-  const T* const kp = reinterpret_cast<const T*>(A.k) + (int64_t)h * dk;
-  const T* const qp = reinterpret_cast<const T*>(A.q) + (int64_t)h * dk;
+  const TQ* const kp = reinterpret_cast<const TQ*>(A.k) + (int64_t)h * dk;
+  const TQ* const qp = reinterpret_cast<const TQ*>(A.q) + (int64_t)h * dk;
   const T* const vp = reinterpret_cast<const T*>(A.v) + (int64_t)h * dv;
   const int st = tid / (DKP / 8), si = (tid % (DKP / 8)) * 8;          // this thread's token of a tile and its eight keys there
-  Raw8<T> rk, rq, rv[NVV];
+  Raw8<TQ> rk, rq;
+  Raw8<T> rv[NVV];
   Raw8<float> rz;
   auto load_tile = [&](int t0) {
     const int nt = min(TT, len - t0);
@@ -341,25 +344,33 @@ __global__ void __launch_bounds__(256) decay_kernel(float* __restrict__ z, int64
   }
 }
 
-template <typename T, int LK, int KPL, bool CHANNEL, int MODE>
+template <typename T, typename TQ, int LK, int KPL, bool CHANNEL, int MODE>
 cudaError_t walk_launch(const LaArgs& A, int n_seqs, cudaStream_t st) {
   constexpr int COLS = kLaThreads / LK * kLaNC, TT = kLaTile / (LK * KPL);
   const size_t smem = (size_t)((1 + (MODE != 1) + (CHANNEL ? 1 : 0)) * kLaTile + TT * COLS) * sizeof(float);
   const dim3 grid((unsigned)((A.dv + COLS - 1) / COLS), (unsigned)A.heads, (unsigned)(MODE == 0 ? n_seqs : n_seqs * A.n_pieces));
-  return launch(walk_kernel<T, LK, KPL, CHANNEL, MODE>, grid, dim3(kLaThreads), smem, st, A);
+  return launch(walk_kernel<T, TQ, LK, KPL, CHANNEL, MODE>, grid, dim3(kLaThreads), smem, st, A);
 }
 
-template <typename T, int LK, int KPL, bool CHANNEL>
+template <typename T, typename TQ, int LK, int KPL, bool CHANNEL>
 cudaError_t scan_launch(const LaArgs& A, int n_seqs, cudaStream_t st) {
-  if (A.n_pieces <= 1) return walk_launch<T, LK, KPL, CHANNEL, 0>(A, n_seqs, st);
-  cudaError_t e = walk_launch<T, LK, KPL, CHANNEL, 1>(A, n_seqs, st);
+  if (A.n_pieces <= 1) return walk_launch<T, TQ, LK, KPL, CHANNEL, 0>(A, n_seqs, st);
+  cudaError_t e = walk_launch<T, TQ, LK, KPL, CHANNEL, 1>(A, n_seqs, st);
   if (e != cudaSuccess) return e;
   const bool v4 = A.vec_s && A.dv % 4 == 0;
   const int64_t per = (int64_t)A.dk * A.dv / (v4 ? 4 : 1);
   const dim3 grid((unsigned)((per + 255) / 256), (unsigned)A.heads, (unsigned)n_seqs);
   e = v4 ? launch(scan_kernel<4>, grid, dim3(256), 0, st, A) : launch(scan_kernel<1>, grid, dim3(256), 0, st, A);
   if (e != cudaSuccess) return e;
-  return walk_launch<T, LK, KPL, CHANNEL, 2>(A, n_seqs, st);
+  return walk_launch<T, TQ, LK, KPL, CHANNEL, 2>(A, n_seqs, st);
+}
+
+// qk_f32: queries and keys are fp32 whatever T is (with fixed decays)
+template <typename T, int LK, int KPL>
+cudaError_t pick_launch(const LaArgs& A, int n_seqs, bool channel, bool qk_f32, cudaStream_t st) {
+  if (channel) return scan_launch<T, T, LK, KPL, true>(A, n_seqs, st);
+  if (qk_f32) return scan_launch<T, float, LK, KPL, false>(A, n_seqs, st);
+  return scan_launch<T, T, LK, KPL, false>(A, n_seqs, st);
 }
 
 int la_cols(int dk) { return kLaThreads / (dk <= 64 ? 8 : dk <= 128 ? 16 : 32) * kLaNC; }
@@ -408,14 +419,15 @@ int b200_linear_attn(const b200_linear_attn_args* a, b200_stream_t stream) {
   B200_CHECK_ARG((int64_t)a->n_seqs * n_pieces <= 65535, "b200_linear_attn: too many pieces");
   const size_t need = b200_linear_attn_workspace_bytes(a->rows, a->max_rows, a->n_seqs, a->heads, a->dk, a->dv);
   B200_CHECK_ARG(need == 0 || (a->workspace && a->workspace_bytes >= need), "b200_linear_attn: workspace too small (%zu of %zu bytes)", a->workspace_bytes, need);
-  const size_t esz = a->dtype == B200_F32 ? 4 : 2;
+  B200_CHECK_ARG(!a->qk_f32 || a->head_decay, "b200_linear_attn: fp32 queries and keys go with fixed decays");
+  const size_t esz = a->dtype == B200_F32 ? 4 : 2, qsz = a->qk_f32 ? 4 : esz;
   auto al = [](const void* p, int64_t bytes) { return ((reinterpret_cast<uintptr_t>(p) | (uintptr_t)bytes) & 15) == 0; };
   float* const ws = (float*)a->workspace;
   const int64_t states = (int64_t)a->n_seqs * n_pieces * a->heads * a->dk * a->dv;
   LaArgs A{a->q, a->k, a->v, a->ldq, a->ldk, a->ldv, a->act, a->q_scale, a->decay_in, a->ld_decay, a->decay_bias, a->decay_in ? 1.0f / a->tau : 0.f, 0,
            a->head_decay, a->state, a->state_slot_stride, a->out, a->ldo, reinterpret_cast<const int4*>(a->seqs), a->heads, a->dk, a->dv, piece, n_pieces,
            ws, ws ? ws + states : nullptr,
-           al(a->q, a->ldq * esz) && al(a->k, a->ldk * esz) && a->dk % 8 == 0, a->decay_in && al(a->decay_in, a->ld_decay * 4) && a->dk % 8 == 0,
+           al(a->q, a->ldq * qsz) && al(a->k, a->ldk * qsz) && a->dk % 8 == 0, a->decay_in && al(a->decay_in, a->ld_decay * 4) && a->dk % 8 == 0,
            al(a->v, a->ldv * esz) && a->dv % 8 == 0, al(a->state, a->state_slot_stride * 4) && al(ws, 0) && a->dv % 4 == 0};
   cudaStream_t st = (cudaStream_t)stream;
   const bool ch = a->decay_in != nullptr;
@@ -428,11 +440,12 @@ int b200_linear_attn(const b200_linear_attn_args* a, b200_stream_t stream) {
                        a->heads * a->dk, A.inv_tau));
       A.z_ready = 1;
     }
-    if (a->dk <= 32) { if (ch) B200_CUDA((scan_launch<T, 8, 4, true>(A, a->n_seqs, st))); else B200_CUDA((scan_launch<T, 8, 4, false>(A, a->n_seqs, st))); }
-    else if (a->dk <= 64) { if (ch) B200_CUDA((scan_launch<T, 8, 8, true>(A, a->n_seqs, st))); else B200_CUDA((scan_launch<T, 8, 8, false>(A, a->n_seqs, st))); }
-    else if (a->dk <= 128) { if (ch) B200_CUDA((scan_launch<T, 16, 8, true>(A, a->n_seqs, st))); else B200_CUDA((scan_launch<T, 16, 8, false>(A, a->n_seqs, st))); }
-    else if (a->dk <= 256) { if (ch) B200_CUDA((scan_launch<T, 32, 8, true>(A, a->n_seqs, st))); else B200_CUDA((scan_launch<T, 32, 8, false>(A, a->n_seqs, st))); }
-    else { if (ch) B200_CUDA((scan_launch<T, 32, 16, true>(A, a->n_seqs, st))); else B200_CUDA((scan_launch<T, 32, 16, false>(A, a->n_seqs, st))); }
+    const bool qf = a->qk_f32 != 0;
+    if (a->dk <= 32) B200_CUDA((pick_launch<T, 8, 4>(A, a->n_seqs, ch, qf, st)));
+    else if (a->dk <= 64) B200_CUDA((pick_launch<T, 8, 8>(A, a->n_seqs, ch, qf, st)));
+    else if (a->dk <= 128) B200_CUDA((pick_launch<T, 16, 8>(A, a->n_seqs, ch, qf, st)));
+    else if (a->dk <= 256) B200_CUDA((pick_launch<T, 32, 8>(A, a->n_seqs, ch, qf, st)));
+    else B200_CUDA((pick_launch<T, 32, 16>(A, a->n_seqs, ch, qf, st)));
   });
   return B200_OK;
 }

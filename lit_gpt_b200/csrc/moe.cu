@@ -2,7 +2,9 @@
 // expert feed-forward over stacked expert weights: y = W_down relu(W_up x)^2 with W_up (E, ff, d), or the gated form
 // y = W_down (silu(W_gate x) * (W_up x)) with the gate and up rows stacked as (E, 2 ff, d); W_down (E, d, ff).
 //
-//  * b200_moe_route: logits, scores, choice and weights in fp32, one CTA per token.
+//  * b200_moe_route: logits, scores, choice and weights in fp32, one CTA per token; optionally the sigmoid gate of a shared expert
+//    from one more row of weights.
+//  * b200_moe_route_logits: choice and weights (softmax among the chosen) from logits a matrix product left, one warp per token.
 //  * b200_moe_plan: counting sort of the (token, choice) pairs by expert -> contiguous row ranges per expert.
 //  * b200_moe_gemm: grouped matrix product over those ranges (one launch for all experts, no host round trip), any
 //    sizes, bf16 or fp32 operands, fp32 accumulation; optional gather of the input rows and relu^2 epilogue.
@@ -38,7 +40,7 @@ template <typename T>
 __global__ void __launch_bounds__(kRtThreads) moe_route_kernel(const T* __restrict__ x, const T* __restrict__ w_router,
                                                                 const T* __restrict__ correction, int* __restrict__ ids,
                                                                 float* __restrict__ wts, int d, int n_expert, int top, int n_group,
-                                                                int keep, int flags) {
+                                                                int keep, int flags, const T* __restrict__ gate_w, float* __restrict__ gate) {
   extern __shared__ float rt_smem[];
   griddep_launch();
   griddep_wait();
@@ -48,9 +50,11 @@ __global__ void __launch_bounds__(kRtThreads) moe_route_kernel(const T* __restri
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int64_t t = blockIdx.x;
   const T* xr = x + t * d;
-  for (int e = warp; e < n_expert; e += kRtThreads / 32) {
-    const float z = warp_dot(xr, w_router + (int64_t)e * d, d, lane);
-    if (lane == 0) {
+  for (int e = warp; e < n_expert + (gate_w ? 1 : 0); e += kRtThreads / 32) {
+    const float z = warp_dot(xr, e < n_expert ? w_router + (int64_t)e * d : gate_w, d, lane);
+    if (lane == 0 && e == n_expert) {
+      gate[t] = 1.0f / (1.0f + expf(-z));
+    } else if (lane == 0) {
       const float corr = correction ? load_as_float(correction, e) : 0.f;
       const float zz = (flags & B200_ROUTE_BIAS) ? z + corr : z;     // a bias is part of the logit; a correction only steers the choice
       const float s = (flags & (B200_ROUTE_SOFTMAX | B200_ROUTE_TOPK_SOFTMAX)) ? zz : 1.0f / (1.0f + expf(-zz));
@@ -114,6 +118,38 @@ __global__ void __launch_bounds__(kRtThreads) moe_route_kernel(const T* __restri
     for (int k = 0; k < top; ++k) sum += expf(score[ids[t * top + k]] - mx);
     for (int k = 0; k < top; ++k) wts[t * top + k] = expf(score[ids[t * top + k]] - mx) / sum;
   }
+}
+
+// The `top` largest of each row's first n_expert logits with softmax weights among them; with `gate`, the sigmoid of column n_expert.
+// One warp per token, top <= 32.
+constexpr int kRlWarps = 4;
+
+__global__ void __launch_bounds__(kRlWarps * 32) moe_route_logits_kernel(const float* __restrict__ logits, int64_t ld, int* __restrict__ ids,
+                                                                         float* __restrict__ wts, float* __restrict__ gate, int64_t tokens, int n_expert, int top) {
+  extern __shared__ float rl_smem[];
+  griddep_launch();
+  griddep_wait();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int64_t t = (int64_t)blockIdx.x * kRlWarps + warp;
+  if (t >= tokens) return;
+  float* const z = rl_smem + warp * n_expert;
+  const float* row = logits + t * ld;
+  for (int e = lane; e < n_expert; e += 32) z[e] = row[e];
+  if (gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-row[n_expert]));
+  __syncwarp();
+  float mine = -INFINITY, best = 0.f;   // lane k holds the k-th chosen logit
+  for (int k = 0; k < top; ++k) {
+    const int e = warp_argmax(z, n_expert, lane);
+    const float v = z[e];
+    if (k == 0) best = v;
+    if (lane == k) { mine = v; ids[t * top + k] = e; }
+    __syncwarp();
+    if (lane == 0) z[e] = -INFINITY;
+    __syncwarp();
+  }
+  const float p = lane < top ? expf(mine - best) : 0.f;
+  const float sum = warp_sum(p);
+  if (lane < top) wts[t * top + lane] = p / sum;
 }
 
 // One CTA.  counts -> expert_off[E + 1] (rows), tile_off[E + 1] (row tiles of `tile_rows`), slot_token[slot] = token,
@@ -232,13 +268,90 @@ __global__ void __launch_bounds__(kGmThreads) moe_gemm_kernel(const T* __restric
 // decode: hidden[p, f] = relu(W_up[ids[p]][f, :] . x[p / top, :])^2 for the pair p = t * top + k; one warp per f.
 // GATED: W_up holds 2 ff rows per expert and hidden[p, f] = silu(row f . x) * (row ff + f . x).
 // limit > 0: the clamped form g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).
+// A gated shared expert that every token uses (sh.up given): blocks beyond the pairs take kShTok tokens each, so that its weights are
+// read once for that many tokens; its products and outputs take the matrix-product dtype as the routed experts' do.
+constexpr int kShTok = 8;
+struct SharedExpert {
+  const void* up; const void* down;   // (2 ff, d), (d, ff)
+  void* hidden; void* out;            // (tokens, ff), (tokens, d)
+  int ff, tokens;
+};
+
+// dot products of one or two weight rows with up to kShTok token rows (row pitch n); every lane gets the sums
+template <typename T, int NW>
+__device__ __forceinline__ void shared_dots(const T* __restrict__ w, int64_t w_pitch, const T* __restrict__ x, int n, int nt, int lane, float (&acc)[NW][kShTok]) {
+#pragma unroll
+  for (int r = 0; r < NW; ++r)
+#pragma unroll
+    for (int t = 0; t < kShTok; ++t) acc[r][t] = 0.f;
+  bool vec = vec8_ok(n, w, x);
+  if (NW > 1) vec = vec && vec8_ok(w_pitch, w);
+  if (vec) {
+#pragma unroll 2
+    for (int i = lane * 8; i < n; i += 256) {
+      float a[NW][8];
+#pragma unroll
+      for (int r = 0; r < NW; ++r) load8(w + r * w_pitch + i, a[r]);
+#pragma unroll
+      for (int t = 0; t < kShTok; ++t) {
+        if (t >= nt) break;
+        float v[8];
+        load8(x + (int64_t)t * n + i, v);
+#pragma unroll
+        for (int r = 0; r < NW; ++r)
+#pragma unroll
+          for (int j = 0; j < 8; ++j) acc[r][t] = fmaf(a[r][j], v[j], acc[r][t]);
+      }
+    }
+  } else {
+    for (int i = lane; i < n; i += 32) {
+      float a[NW];
+#pragma unroll
+      for (int r = 0; r < NW; ++r) a[r] = load_as_float(w, r * w_pitch + i);
+#pragma unroll
+      for (int t = 0; t < kShTok; ++t) {
+        if (t >= nt) break;
+        const float v = load_as_float(x, (int64_t)t * n + i);
+#pragma unroll
+        for (int r = 0; r < NW; ++r) acc[r][t] = fmaf(a[r], v, acc[r][t]);
+      }
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < kShTok; ++t) {
+    if (t >= nt) break;
+#pragma unroll
+    for (int r = 0; r < NW; ++r) acc[r][t] = warp_sum(acc[r][t]);
+  }
+}
+
+template <typename T>
+__device__ __forceinline__ float as_dtype(float v) {   // v rounded to T
+  T r;
+  store_from_float(&r, 0, v);
+  return load_as_float(&r, 0);
+}
+
 template <typename T, bool GATED>
 __global__ void __launch_bounds__(256) moe_gemv_up_kernel(const T* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ w_up,
-                                                          T* __restrict__ hidden, int top, int d, int ff, float limit, float alpha) {
+                                                          T* __restrict__ hidden, int pairs, int top, int d, int ff, float limit, float alpha, SharedExpert sh) {
   griddep_launch();
   griddep_wait();
   const int p = blockIdx.y, lane = threadIdx.x & 31;
   const int f = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (GATED && p >= pairs) {
+    if (f >= sh.ff) return;
+    const int t0 = (p - pairs) * kShTok, nt = min(kShTok, sh.tokens - t0);
+    float acc[2][kShTok];
+    shared_dots<T, 2>(reinterpret_cast<const T*>(sh.up) + (int64_t)f * d, (int64_t)sh.ff * d, x + (int64_t)t0 * d, d, nt, lane, acc);
+#pragma unroll
+    for (int t = 0; t < kShTok; ++t) {
+      if (t >= nt || lane != t) continue;
+      const float g = as_dtype<T>(acc[0][t]);
+      store_from_float(reinterpret_cast<T*>(sh.hidden), (int64_t)(t0 + t) * sh.ff + f, g / (1.0f + expf(-g)) * as_dtype<T>(acc[1][t]));
+    }
+    return;
+  }
   if (f >= ff) return;
   const T* xr = x + (int64_t)(p / top) * d;
   if (GATED) {
@@ -271,12 +384,21 @@ __global__ void __launch_bounds__(256) moe_gemv_up_kernel(const T* __restrict__ 
 template <typename T>
 __global__ void __launch_bounds__(256) moe_gemv_down_kernel(const T* __restrict__ hidden, const int* __restrict__ ids,
                                                             const float* __restrict__ wts, const T* __restrict__ w_down,
-                                                            T* __restrict__ out, int top, int d, int ff) {
+                                                            T* __restrict__ out, int tokens, int top, int d, int ff, SharedExpert sh) {
   griddep_launch();
   griddep_wait();
   const int t = blockIdx.y, lane = threadIdx.x & 31;
   const int c = blockIdx.x * 8 + (threadIdx.x >> 5);
   if (c >= d) return;
+  if (t >= tokens) {
+    const int t0 = (t - tokens) * kShTok, nt = min(kShTok, sh.tokens - t0);
+    float acc[1][kShTok];
+    shared_dots<T, 1>(reinterpret_cast<const T*>(sh.down) + (int64_t)c * sh.ff, 0, reinterpret_cast<const T*>(sh.hidden) + (int64_t)t0 * sh.ff, sh.ff, nt, lane, acc);
+#pragma unroll
+    for (int i = 0; i < kShTok; ++i)
+      if (i < nt && lane == i) store_from_float(reinterpret_cast<T*>(sh.out), (int64_t)(t0 + i) * d + c, acc[0][i]);
+    return;
+  }
   float total = 0.f;
   for (int k = 0; k < top; ++k) {
     const int p = t * top + k;
@@ -326,15 +448,25 @@ using namespace b200;
 extern "C" {
 
 int b200_moe_route(const void* x, const void* w_router, const void* correction, int32_t* ids, float* weights, int64_t tokens, int d,
-                   int n_expert, int top, int n_group, int keep, int flags, int dtype, b200_stream_t stream) {
-  B200_CHECK_ARG(x && w_router && ids && weights, "b200_moe_route: null pointer");
+                   int n_expert, int top, int n_group, int keep, int flags, const void* gate_w, float* gate, int dtype, b200_stream_t stream) {
+  B200_CHECK_ARG(x && w_router && ids && weights && !gate_w == !gate, "b200_moe_route: null pointer");
   B200_CHECK_ARG(tokens > 0 && tokens <= 0x7fffffff && d > 0 && n_expert > 0 && top > 0 && top <= n_expert, "b200_moe_route: bad shape");
   B200_CHECK_ARG(n_group > 0 && n_expert % n_group == 0 && keep > 0 && keep <= n_group, "b200_moe_route: groups must divide the experts");
   B200_CHECK_ARG((int64_t)keep * (n_expert / n_group) >= top, "b200_moe_route: the kept groups hold fewer experts than are chosen");
   const size_t smem = (size_t)(2 * n_expert + n_group) * sizeof(float);
   B200_CHECK_ARG(smem <= 48 * 1024, "b200_moe_route: too many experts");
   B200_FLOAT_TYPES(dtype, T, B200_CUDA(launch(moe_route_kernel<T>, dim3((unsigned)tokens), dim3(kRtThreads), smem, (cudaStream_t)stream, (const T*)x,
-                                               (const T*)w_router, (const T*)correction, ids, weights, d, n_expert, top, n_group, keep, flags)));
+                                               (const T*)w_router, (const T*)correction, ids, weights, d, n_expert, top, n_group, keep, flags, (const T*)gate_w, gate)));
+  return B200_OK;
+}
+
+int b200_moe_route_logits(const float* logits, int64_t ld, int32_t* ids, float* weights, float* gate, int64_t tokens, int n_expert, int top,
+                          b200_stream_t stream) {
+  B200_CHECK_ARG(logits && ids && weights && tokens > 0 && tokens <= 0x7fffffff, "b200_moe_route_logits: bad argument");
+  B200_CHECK_ARG(n_expert > 0 && top > 0 && top <= n_expert && top <= 32 && n_expert <= 3072 && ld >= n_expert + (gate ? 1 : 0),
+                 "b200_moe_route_logits: at most 32 of at most 3072 experts");
+  B200_CUDA(launch(moe_route_logits_kernel, dim3((unsigned)((tokens + kRlWarps - 1) / kRlWarps)), dim3(kRlWarps * 32),
+                   (size_t)kRlWarps * n_expert * sizeof(float), (cudaStream_t)stream, logits, ld, ids, weights, gate, tokens, n_expert, top));
   return B200_OK;
 }
 
@@ -365,21 +497,25 @@ int b200_moe_gemm(const void* a, int64_t lda, const int32_t* row_src, const void
 }
 
 int b200_moe_gemv(const void* x, const int32_t* ids, const float* weights, const void* w_up, const void* w_down, void* hidden, void* out,
-                  int64_t tokens, int top, int d, int ff, int gated, float limit, float alpha, int dtype, b200_stream_t stream) {
+                  int64_t tokens, int top, int d, int ff, int gated, float limit, float alpha, const void* shared_up, const void* shared_down,
+                  int shared_ff, void* shared_hidden, void* shared_out, int dtype, b200_stream_t stream) {
+  B200_CHECK_ARG(!shared_up || (gated == 1 && shared_down && shared_hidden && shared_out && shared_ff > 0), "b200_moe_gemv: a shared expert goes with gated 1");
   B200_CHECK_ARG(x && ids && weights && w_up && w_down && hidden && out, "b200_moe_gemv: null pointer");
   B200_CHECK_ARG(gated >= 0 && gated <= 2 && (gated != 2 || limit > 0.f), "b200_moe_gemv: gated is 0 (relu^2), 1 (silu gate) or 2 (clamped gate, limit > 0)");
   if (gated != 2) limit = 0.f;
   B200_CHECK_ARG(tokens > 0 && tokens * top <= 65535 && d > 0 && ff > 0, "b200_moe_gemv: bad shape");
   cudaStream_t st = (cudaStream_t)stream;
+  const SharedExpert sh{shared_up, shared_down, shared_hidden, shared_out, shared_up ? shared_ff : 0, (int)tokens};
+  const int pairs = (int)(tokens * top), extra = shared_up ? (int)((tokens + kShTok - 1) / kShTok) : 0, ffm = shared_ff > ff && shared_up ? shared_ff : ff;
   B200_FLOAT_TYPES(dtype, T, {
     if (gated)
-      B200_CUDA(launch(moe_gemv_up_kernel<T, true>, dim3((unsigned)((ff + 7) / 8), (unsigned)(tokens * top)), dim3(256), 0, st, (const T*)x, ids,
-                       (const T*)w_up, (T*)hidden, top, d, ff, limit, alpha));
+      B200_CUDA(launch(moe_gemv_up_kernel<T, true>, dim3((unsigned)((ffm + 7) / 8), (unsigned)(pairs + extra)), dim3(256), 0, st, (const T*)x, ids,
+                       (const T*)w_up, (T*)hidden, pairs, top, d, ff, limit, alpha, sh));
     else
-      B200_CUDA(launch(moe_gemv_up_kernel<T, false>, dim3((unsigned)((ff + 7) / 8), (unsigned)(tokens * top)), dim3(256), 0, st, (const T*)x, ids,
-                       (const T*)w_up, (T*)hidden, top, d, ff, limit, alpha));
-    B200_CUDA(launch(moe_gemv_down_kernel<T>, dim3((unsigned)((d + 7) / 8), (unsigned)tokens), dim3(256), 0, st, (const T*)hidden, ids, weights,
-                     (const T*)w_down, (T*)out, top, d, ff));
+      B200_CUDA(launch(moe_gemv_up_kernel<T, false>, dim3((unsigned)((ff + 7) / 8), (unsigned)pairs), dim3(256), 0, st, (const T*)x, ids,
+                       (const T*)w_up, (T*)hidden, pairs, top, d, ff, limit, alpha, sh));
+    B200_CUDA(launch(moe_gemv_down_kernel<T>, dim3((unsigned)((d + 7) / 8), (unsigned)(tokens + extra)), dim3(256), 0, st, (const T*)hidden, ids, weights,
+                     (const T*)w_down, (T*)out, (int)tokens, top, d, ff, sh));
   });
   return B200_OK;
 }

@@ -341,6 +341,20 @@ template <typename T>
 __global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ in, T* __restrict__ out, int64_t rows, int ff, int kind) {
   griddep_launch();
   griddep_wait();
+  if (vec8_ok(ff, in, out)) {
+    const int per = ff / 8;
+    const int64_t n8 = rows * per;
+    for (int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x; i < n8; i += (int64_t)gridDim.x * 256) {
+      const int64_t r = i / per, c = (i - r * per) * 8;
+      float g[8], u[8];
+      load8(in + r * 2 * ff + c, g);
+      load8(in + r * 2 * ff + ff + c, u);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) g[j] = activate(g[j], kind) * u[j];
+      store8(out + r * ff + c, g);
+    }
+    return;
+  }
   const int64_t n = rows * ff;
   for (int64_t i = (int64_t)blockIdx.x * 256 + threadIdx.x; i < n; i += (int64_t)gridDim.x * 256) {
     const int64_t r = i / ff, c = i - r * ff;
@@ -512,6 +526,107 @@ __global__ void __launch_bounds__(256) scaled_residual_kernel(ScaledResidualArgs
       if constexpr (V == 8) store8(reinterpret_cast<T*>(A.act) + o, x);
       else store_from_float(reinterpret_cast<T*>(A.act), o, x[0]);
     }
+  }
+}
+
+// Residual update of a pre-normed block whose sublayers are scaled per channel, fused with the RMS norm that feeds the next sublayer:
+//   y    = y0[row]  |  sum_k wts[row, k] * y0[slot_of[row, k]]      (the routed experts' rows, weighted here instead of in a pass of its own)
+//   x   += mult * scale * (y + gate[row] * y1[row])                 (fp32 stream; y1, gate, scale optional)
+//   act  = T(x / sqrt(mean(x^2) + eps) * (w or 1 + w))              (skipped without w)
+// One CTA per row.  Whole rows of up to R * 1024 numbers stay in registers between the two passes; others are read back.
+struct GatedResidualArgs {
+  const void* y0; const int* slot_of; const float* wts; int top;
+  const void* y1; const float* gate; const void* scale; float mult;
+  float* x; const void* w; int plus_one; void* act;
+  int d;
+  float eps;
+};
+
+template <typename T, int V>
+__device__ __forceinline__ void gated_branch(const GatedResidualArgs& A, int64_t row, float gate, int i, float (&y)[V]) {
+  const T* y0 = reinterpret_cast<const T*>(A.y0);
+  auto ld = [](const T* p, float (&f)[V]) {
+    if constexpr (V == 8) load8(p, f);
+    else f[0] = load_as_float(p, 0);
+  };
+  if (A.slot_of) {
+#pragma unroll
+    for (int j = 0; j < V; ++j) y[j] = 0.f;
+    for (int k = 0; k < A.top; ++k) {
+      float t[V];
+      const float w = A.wts[row * A.top + k];
+      ld(y0 + (int64_t)A.slot_of[row * A.top + k] * A.d + i, t);
+#pragma unroll
+      for (int j = 0; j < V; ++j) y[j] = fmaf(w, t[j], y[j]);
+    }
+  } else {
+    ld(y0 + row * A.d + i, y);
+  }
+  if (A.y1) {
+    float t[V];
+    ld(reinterpret_cast<const T*>(A.y1) + row * A.d + i, t);
+#pragma unroll
+    for (int j = 0; j < V; ++j) y[j] = fmaf(gate, t[j], y[j]);
+  }
+  if (A.scale) {
+    float t[V];
+    ld(reinterpret_cast<const T*>(A.scale) + i, t);
+#pragma unroll
+    for (int j = 0; j < V; ++j) y[j] *= t[j];
+  }
+}
+
+template <typename T, int R>   // R = 0: any size
+__global__ void __launch_bounds__(kRowThreads) gated_residual_kernel(GatedResidualArgs A) {
+  __shared__ float s_part[kRowThreads / 32];
+  griddep_launch();
+  griddep_wait();
+  const int64_t row = blockIdx.x;
+  const int d = A.d;
+  float* const xr = A.x + row * d;
+  T* const ar = reinterpret_cast<T*>(A.act) + row * d;
+  const T* const w = reinterpret_cast<const T*>(A.w);
+  const float gate = A.gate ? A.gate[row] : 1.0f, one = A.plus_one ? 1.0f : 0.0f;
+  float ss = 0.f;
+  if constexpr (R > 0) {
+    float x[R][8];
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int i = (r * kRowThreads + threadIdx.x) * 8;
+      if (i >= d) break;
+      float y[8];
+      load8(xr + i, x[r]);
+      gated_branch<T, 8>(A, row, gate, i, y);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        x[r][j] = fmaf(A.mult, y[j], x[r][j]);
+        ss = fmaf(x[r][j], x[r][j], ss);
+      }
+      store8(xr + i, x[r]);
+    }
+    if (!w) return;
+    const float rstd = 1.0f / sqrtf(cta_sum(ss, s_part) / (float)d + A.eps);
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int i = (r * kRowThreads + threadIdx.x) * 8;
+      if (i >= d) break;
+      float g[8];
+      load8(w + i, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) g[j] = x[r][j] * rstd * (g[j] + one);
+      store8(ar + i, g);
+    }
+  } else {
+    for (int i = threadIdx.x; i < d; i += kRowThreads) {   // each thread reads back only what it wrote itself
+      float y[1];
+      gated_branch<T, 1>(A, row, gate, i, y);
+      const float v = fmaf(A.mult, y[0], xr[i]);
+      ss = fmaf(v, v, ss);
+      xr[i] = v;
+    }
+    if (!w) return;
+    const float rstd = 1.0f / sqrtf(cta_sum(ss, s_part) / (float)d + A.eps);
+    for (int i = threadIdx.x; i < d; i += kRowThreads) store_from_float(ar, i, xr[i] * rstd * (load_as_float(w, i) + one));
   }
 }
 
@@ -712,6 +827,26 @@ int b200_scaled_residual(const b200_scaled_residual_args* a, b200_stream_t strea
   B200_FLOAT_TYPES(a->dtype, T, {
     if (vec) B200_CUDA(launch(scaled_residual_kernel<T, 8>, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, A));
     else B200_CUDA(launch(scaled_residual_kernel<T, 1>, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, A));
+  });
+  return B200_OK;
+}
+
+int b200_gated_residual(const b200_gated_residual_args* a, b200_stream_t stream) {
+  B200_CHECK_ARG(a && a->x && a->y0 && a->rows > 0 && a->rows <= 0x7fffffff && a->d > 0, "b200_gated_residual: bad argument");
+  B200_CHECK_ARG(!a->slot_of || (a->wts && a->top > 0), "b200_gated_residual: gathered rows need their weights");
+  B200_CHECK_ARG(!a->w || a->act, "b200_gated_residual: the norm needs somewhere to go");
+  const GatedResidualArgs A{a->y0, a->slot_of, a->wts, a->top, a->y1, a->gate, a->scale, a->mult, a->x, a->w, a->plus_one, a->act, a->d, a->eps};
+  auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool vec = a->d % 8 == 0 && al(a->y0) && al(a->y1) && al(a->scale) && al(a->x) && al(a->w) && al(a->act);
+  const int per = kRowThreads * 8;
+  const dim3 grid((unsigned)a->rows), block(kRowThreads);
+  cudaStream_t st = (cudaStream_t)stream;
+  B200_FLOAT_TYPES(a->dtype, T, {
+    if (vec && a->d <= per) B200_CUDA(launch(gated_residual_kernel<T, 1>, grid, block, 0, st, A));
+    else if (vec && a->d <= 2 * per) B200_CUDA(launch(gated_residual_kernel<T, 2>, grid, block, 0, st, A));
+    else if (vec && a->d <= 4 * per) B200_CUDA(launch(gated_residual_kernel<T, 4>, grid, block, 0, st, A));
+    else if (vec && a->d <= 8 * per) B200_CUDA(launch(gated_residual_kernel<T, 8>, grid, block, 0, st, A));
+    else B200_CUDA(launch(gated_residual_kernel<T, 0>, grid, block, 0, st, A));
   });
   return B200_OK;
 }

@@ -9,33 +9,31 @@
 //             frequencies in fp64 and reduced to [-pi, pi] before the fp32 sine and cosine
 //   the other dimensions pass unchanged.
 //
-// Up to three groups of heads (e.g. queries, keys, values of one fused projection) run as one launch; one CTA per (row, group).
+// Up to four groups of heads (e.g. the queries and keys of two mixers that share one fused projection) run as one launch; one CTA per (row,
+// group).  A group may be written in fp32 whatever the dtype it is read in (operands of an fp32 recurrence).
 #include "common.cuh"
 
 namespace b200 {
 
 namespace {
 
-constexpr int kHrThreads = 128, kHrMaxSegs = 3;
+constexpr int kHrThreads = 128, kHrMaxSegs = 4;
 
 struct HeadSeg {
   const void* in; void* out; const void* norm_w; const void* freq; const int64_t* out_rows;
   int64_t ld_in, ld_out;
   int heads, dim, in_stride, out_stride, rot_off, rot_dims, interleaved;
   float mag;
-  int norm_all, freq_f64;
+  int norm_all, freq_f64, out_f32;
 };
 struct HeadSegs { HeadSeg s[kHrMaxSegs]; };
 
 // grid (rows, groups): the CTA of a row works out the row's cosines and sines once (they depend on the position and the pair only, not
 // on the head), then its warps take the heads of the group in turn
-template <typename T>
-__global__ void __launch_bounds__(kHrThreads) head_rope_kernel(HeadSegs S, const int* __restrict__ row_pos, float eps) {
+template <typename T, typename TO>
+__device__ __forceinline__ void head_rope_row(const HeadSeg& s, const int* __restrict__ row_pos, float eps) {
   extern __shared__ __align__(16) float hr_smem[];   // [rot_dims / 2] cosines, then as many sines, both times mag
   __shared__ float s_part[kHrThreads / 32];
-  griddep_launch();
-  griddep_wait();
-  const HeadSeg s = S.s[blockIdx.y];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int64_t row = blockIdx.x;
   const int64_t orow = s.out_rows ? s.out_rows[row] : row;
@@ -86,7 +84,7 @@ __global__ void __launch_bounds__(kHrThreads) head_rope_kernel(HeadSegs S, const
   }
   for (int h = warp; h < s.heads; h += kHrThreads / 32) {
     const T* x = reinterpret_cast<const T*>(s.in) + row * s.ld_in + (int64_t)h * s.in_stride;
-    T* o = reinterpret_cast<T*>(s.out) + orow * s.ld_out + (int64_t)h * s.out_stride;
+    TO* o = reinterpret_cast<TO*>(s.out) + orow * s.ld_out + (int64_t)h * s.out_stride;
     const T* w = s.norm_all ? wall + (int64_t)h * s.dim : wall;
     float rstd = rstd_all;
     if (w && !s.norm_all) {
@@ -113,6 +111,15 @@ __global__ void __launch_bounds__(kHrThreads) head_rope_kernel(HeadSegs S, const
   }
 }
 
+template <typename T>
+__global__ void __launch_bounds__(kHrThreads) head_rope_kernel(HeadSegs S, const int* __restrict__ row_pos, float eps) {
+  griddep_launch();
+  griddep_wait();
+  const HeadSeg s = S.s[blockIdx.y];
+  if (s.out_f32) head_rope_row<T, float>(s, row_pos, eps);
+  else head_rope_row<T, T>(s, row_pos, eps);
+}
+
 }  // namespace
 
 }  // namespace b200
@@ -122,7 +129,7 @@ using namespace b200;
 extern "C" {
 
 int b200_head_rope(const b200_head_rope_seg* segs, int n_segs, const int32_t* row_pos, int64_t rows, float eps, int dtype, b200_stream_t stream) {
-  B200_CHECK_ARG(segs && n_segs >= 1 && n_segs <= kHrMaxSegs && row_pos, "b200_head_rope: one to three groups of heads and the rows' positions");
+  B200_CHECK_ARG(segs && n_segs >= 1 && n_segs <= kHrMaxSegs && row_pos, "b200_head_rope: one to four groups of heads and the rows' positions");
   B200_CHECK_ARG(rows > 0 && rows <= 0x7fffffff, "b200_head_rope: bad row count");
   HeadSegs S;
   int max_rot = 0;
@@ -133,7 +140,7 @@ int b200_head_rope(const b200_head_rope_seg* segs, int n_segs, const int32_t* ro
                    "b200_head_rope: the rotated dimensions must be an even run inside the head, with their frequencies");
     B200_CHECK_ARG(!a.norm_all || (a.norm_w && (a.in_stride == a.dim || a.heads == 1)), "b200_head_rope: a norm over all heads needs its weight and heads side by side");
     S.s[i] = HeadSeg{a.in, a.out, a.norm_w, a.freq, a.out_rows, a.ld_in, a.ld_out, a.heads, a.dim, a.in_stride, a.out_stride, a.rot_off, a.rot_dims,
-                     a.interleaved, a.mag, a.norm_all, a.freq_f64};
+                     a.interleaved, a.mag, a.norm_all, a.freq_f64, a.out_f32};
     if (i < n_segs) max_rot = a.rot_dims > max_rot ? a.rot_dims : max_rot;
   }
   B200_CHECK_ARG(max_rot <= 8192, "b200_head_rope: at most 8192 rotated dimensions");

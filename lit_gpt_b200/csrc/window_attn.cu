@@ -47,6 +47,7 @@ struct WaArgs {
   int64_t ldg;
   int gate_mode;                    // 1: column h of the gate row; 2: column h * dv + c
   int keep;                         // first positions that never leave the window, nor the cache
+  float out_scale;                  // factor of the output
   float cap_log2, inv_cap;          // soft cap: cap * log2(e), and 1 / (cap * log2(e)); inv_cap 0: none
 };
 
@@ -226,7 +227,7 @@ __global__ void __launch_bounds__(kWaThreads) window_attn_kernel(WaArgs A) {
 #pragma unroll
     for (int b = 0; b < 8; ++b) {
       const int cc = (b < 4 ? 0 : 64) + 4 * tx + (b & 3);
-      if (cc < dvc) store_from_float(orow, cc, o[a][b] * inv * wa_gate<T>(A, first + i, h, c0 + cc));
+      if (cc < dvc) store_from_float(orow, cc, o[a][b] * inv * A.out_scale * wa_gate<T>(A, first + i, h, c0 + cc));
     }
   }
 }
@@ -402,7 +403,7 @@ __global__ void __launch_bounds__(kWdThreads) window_decode_kernel(WaArgs A) {
   for (int c = tid; c < dv; c += kWdThreads) {
     float t = 0.f;
     for (int r = 0; r < vrows; ++r) t += part[r * dv + c];
-    store_from_float(reinterpret_cast<T*>(A.out), (int64_t)row * A.ldo + (int64_t)h * dv + c, t * inv * wa_gate<T>(A, row, h, c));
+    store_from_float(reinterpret_cast<T*>(A.out), (int64_t)row * A.ldo + (int64_t)h * dv + c, t * inv * A.out_scale * wa_gate<T>(A, row, h, c));
   }
   // The row's own key and value enter the ring here: they replace position pos - ring (kept rows are never replaced), which no row of this step can see
   // (ring >= window), and every CTA reads the current position from the step's rows, never from the ring.
@@ -458,7 +459,8 @@ int b200_window_attn(const b200_window_attn_args* a, b200_stream_t stream) {
   B200_CHECK_ARG(a->gate_mode >= 0 && a->gate_mode <= 2 && (a->gate_mode == 0 || a->gate), "b200_window_attn: bad gate");
   const WaArgs A{a->q, a->k, a->v, a->out, a->ldq, a->ldk, a->ldv, a->ldo, a->k_ring, a->v_ring, a->sink, reinterpret_cast<const int4*>(a->seqs),
                  a->ring, a->n_head, a->n_kv_head, a->dk, a->dv, a->window, a->scale * kLog2e, a->row_seq != nullptr,
-                 a->dist_r1, a->dist_r2, a->gate_mode ? a->gate : nullptr, a->ldg, a->gate_mode, a->keep, a->softcap * kLog2e,
+                 a->dist_r1, a->dist_r2, a->gate_mode ? a->gate : nullptr, a->ldg, a->gate_mode, a->keep, a->out_scale,
+                 a->softcap * kLog2e,
                  a->softcap > 0.f ? 1.0f / (a->softcap * kLog2e) : 0.f};
   cudaStream_t st = (cudaStream_t)stream;
   const size_t esz = a->dtype == B200_F32 ? 4 : 2;

@@ -758,20 +758,37 @@ def latent_decode_tune(force_any_size_kernel: bool = False) -> bool:
 
 
 def moe_route(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], top: int, n_group: int, keep: int,
-              softmax: bool = False, group_max: bool = False, topk_softmax: bool = False, bias: bool = False):
+              softmax: bool = False, group_max: bool = False, topk_softmax: bool = False, bias: bool = False, gate_w: Optional[torch.Tensor] = None):
     """-> (ids int32 (n, top), weights fp32 (n, top)); see b200_moe_route.  softmax: scores are a softmax over all experts
     instead of sigmoids; group_max: a group ranks by its largest score instead of the sum of its two largest; topk_softmax: the
-    largest raw logits are chosen and weighted by a softmax among those few; bias: `correction` is a bias inside the logit."""
-    C.require_cuda(x, w_router, correction)
+    largest raw logits are chosen and weighted by a softmax among those few; bias: `correction` is a bias inside the logit.
+    gate_w (d numbers): a third result, fp32 (n,) = sigmoid(x . gate_w), the gate of a shared expert."""
+    C.require_cuda(x, w_router, correction, gate_w)
     n, d = x.shape
     E = w_router.shape[0]
     ids = torch.empty((n, top), dtype=torch.int32, device=x.device)
     wts = torch.empty((n, top), dtype=torch.float32, device=x.device)
+    gate = torch.empty(n, dtype=torch.float32, device=x.device) if gate_w is not None else None
     C.check(C.load_core().b200_moe_route(x.data_ptr(), w_router.data_ptr(), C.ptr(correction), ids.data_ptr(), wts.data_ptr(), n, d, E, top, n_group,
                                          keep, (C.ROUTE_SOFTMAX if softmax else 0) | (C.ROUTE_GROUP_MAX if group_max else 0)
-                                         | (C.ROUTE_TOPK_SOFTMAX if topk_softmax else 0) | (C.ROUTE_BIAS if bias else 0), _code(x),
-                                         C.stream_ptr(x.device)), "moe_route")
-    return ids, wts
+                                         | (C.ROUTE_TOPK_SOFTMAX if topk_softmax else 0) | (C.ROUTE_BIAS if bias else 0), C.ptr(gate_w),
+                                         C.ptr(gate), _code(x), C.stream_ptr(x.device)), "moe_route")
+    return (ids, wts) if gate is None else (ids, wts, gate)
+
+
+def moe_route_logits(logits: torch.Tensor, experts: int, top: int, gate: bool = False):
+    """The `top` <= 32 largest of each row's first `experts` logits (fp32 (n, columns)) -> ids int32 (n, top), softmax weights among them
+    fp32 (n, top), and with `gate` the sigmoid of column `experts`, fp32 (n,)."""
+    C.require_cuda(logits)
+    if logits.dtype != torch.float32 or logits.stride(-1) != 1:
+        raise C.B200Error("moe_route_logits: fp32 logits with unit inner stride")
+    n = logits.shape[0]
+    ids = torch.empty((n, top), dtype=torch.int32, device=logits.device)
+    wts = torch.empty((n, top), dtype=torch.float32, device=logits.device)
+    g = torch.empty(n, dtype=torch.float32, device=logits.device) if gate else None
+    C.check(C.load_core().b200_moe_route_logits(logits.data_ptr(), logits.stride(0), ids.data_ptr(), wts.data_ptr(), C.ptr(g), n, experts, top,
+                                                C.stream_ptr(logits.device)), "moe_route_logits")
+    return (ids, wts, g) if gate else (ids, wts)
 
 
 MOE_GEMV_MAX_PAIRS = 64   # up to this many (token, choice) pairs the experts run as weight-streaming GEMVs
@@ -790,7 +807,8 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_up: tor
     if n * top <= MOE_GEMV_MAX_PAIRS:
         hidden = torch.empty((n * top, ff), dtype=x.dtype, device=x.device)
         C.check(lib.b200_moe_gemv(x.data_ptr(), ids.data_ptr(), wts.data_ptr(), w_up.data_ptr(), w_down.data_ptr(), hidden.data_ptr(), out.data_ptr(),
-                                  n, top, d, ff, (2 if limit > 0 else 1) if gated else 0, float(limit), float(alpha), code, st), "moe_gemv")
+                                  n, top, d, ff, (2 if limit > 0 else 1) if gated else 0, float(limit), float(alpha), None, None, 0, None, None, code, st),
+                "moe_gemv")
         return out
     plan = moe_plan(ids, E)
     up_rows = 2 * ff if gated else ff
@@ -803,6 +821,24 @@ def moe_experts(x: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_up: tor
     C.check(lib.b200_moe_gemm(hidden.data_ptr(), ff, None, w_down.data_ptr(), y.data_ptr(), d, plan.expert_off.data_ptr(), plan.tile_off.data_ptr(),
                               n * top, E, d, ff, 0, code, st), "moe_gemm(down)")
     return moe_combine(y, plan, wts)
+
+
+def moe_experts_shared(x: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, shared_up: torch.Tensor,
+                       shared_down: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Gated experts for a few tokens (at most MOE_GEMV_MAX_PAIRS pairs) together with a shared expert of the same form that every token
+    uses, in the same two launches: -> (weighted sum of the chosen experts, the shared expert's result), both (n, d)."""
+    C.require_cuda(x, ids, wts, w_up, w_down, shared_up, shared_down)
+    n, d = x.shape
+    ff, top, ffs = w_down.shape[2], ids.shape[1], shared_down.shape[1]
+    if n * top > MOE_GEMV_MAX_PAIRS:
+        raise C.B200Error("moe_experts_shared: too many tokens")
+    hidden = torch.empty((n * top, ff), dtype=x.dtype, device=x.device)
+    shidden = torch.empty((n, ffs), dtype=x.dtype, device=x.device)
+    out, sout = torch.empty((n, d), dtype=x.dtype, device=x.device), torch.empty((n, d), dtype=x.dtype, device=x.device)
+    C.check(C.load_core().b200_moe_gemv(x.data_ptr(), ids.data_ptr(), wts.data_ptr(), w_up.data_ptr(), w_down.data_ptr(), hidden.data_ptr(), out.data_ptr(),
+                                        n, top, d, ff, 1, 0.0, 1.0, shared_up.data_ptr(), shared_down.data_ptr(), ffs, shidden.data_ptr(), sout.data_ptr(),
+                                        _code(x), C.stream_ptr(x.device)), "moe_gemv")
+    return out, sout
 
 
 class MoEPlan:
@@ -933,6 +969,30 @@ def scaled_residual(x: torch.Tensor, *, y0: Optional[torch.Tensor] = None, s0: O
     C.check(C.load_core().b200_scaled_residual(ctypes.byref(args), C.stream_ptr(x.device)), "scaled_residual")
 
 
+def gated_residual(x: torch.Tensor, y0: torch.Tensor, eps: float, *, slot_of: Optional[torch.Tensor] = None, wts: Optional[torch.Tensor] = None,
+                   y1: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, scale: Optional[torch.Tensor] = None, mult: float = 1.0,
+                   norm_w: Optional[torch.Tensor] = None, plus_one: bool = False, act: Optional[torch.Tensor] = None) -> None:
+    """x (fp32 (rows, d), in place) += mult * scale * (y + gate[row] * y1); act = T(x / rms(x) * norm_w), or * (1 + norm_w) with plus_one.
+    y: y0 (rows, d), or with slot_of int32 (rows, top) and wts fp32 (rows, top) the weighted sum of y0's rows slot_of[row, k] -- routed
+    experts' rows, combined here instead of in a pass of their own."""
+    C.require_cuda(x, y0, slot_of, wts, y1, gate, scale, norm_w, act)
+    if x.dtype != torch.float32 or not x.is_contiguous() or any(t is not None and (t.dtype != torch.float32 or not t.is_contiguous()) for t in (wts, gate)):
+        raise C.B200Error("gated_residual: the stream, weights and gate must be contiguous fp32")
+    if any(t is not None and (t.dtype != y0.dtype or not t.is_contiguous()) for t in (y0, y1, scale, norm_w, act)):
+        raise C.B200Error("gated_residual: branches, scale, norm and output in one dtype, contiguous")
+    d = x.shape[-1]
+    rows = x.numel() // d
+    top = 0
+    if slot_of is not None:
+        if wts is None or slot_of.dtype != torch.int32 or not slot_of.is_contiguous() or slot_of.numel() != wts.numel() or slot_of.numel() % rows:
+            raise C.B200Error("gated_residual: gathered rows need int32 indices and as many weights")
+        top = slot_of.numel() // rows
+    args = C.GatedResidualArgs(y0=y0.data_ptr(), slot_of=C.ptr(slot_of), wts=C.ptr(wts), top=top, y1=C.ptr(y1), gate=C.ptr(gate), scale=C.ptr(scale),
+                               mult=float(mult), x=x.data_ptr(), w=C.ptr(norm_w), plus_one=int(plus_one), act=C.ptr(act) if norm_w is not None else None,
+                               rows=rows, d=d, eps=float(eps), dtype=_code(y0))
+    C.check(C.load_core().b200_gated_residual(ctypes.byref(args), C.stream_ptr(x.device)), "gated_residual")
+
+
 def conv_group(w: torch.Tensor, out: torch.Tensor, col0: int, heads: int, dim: int, *, act: int = 0, post: int = 0, rot_dims: int = 0,
                inv_freq: Optional[torch.Tensor] = None, rot_mscale: float = 1.0, post_scale: float = 1.0, eps: float = 0.0) -> "C.ConvGroup":
     """One group of heads for ``short_conv``: act 0 none / 1 silu; post 0 none / 1 rotate + RMS norm / 2 unit vector."""
@@ -1001,11 +1061,12 @@ def linear_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.
                 decay_bias: Optional[torch.Tensor] = None, tau: float = 1.0) -> torch.Tensor:
     """Decaying linear attention over the step's rows: per head S <- diag(g) S + k v^T, o = S^T q; state (slots, heads * dk * dv) fp32 is
     read (unless the sequence starts at 0) and written.  q, k (n, heads * dk) and v (n, heads * dv) are raw projections (`silu`: each passes
-    through it; q then times q_scale).  g: head_decay fp32 (heads,), fixed -- or decay_in fp32 (n, heads * dk), raw and used as scratch, with
+    through it; q then times q_scale); with head_decay q and k may also be fp32 beside a 16-bit v.  g: head_decay fp32 (heads,), fixed -- or decay_in fp32 (n, heads * dk), raw and used as scratch, with
     decay_bias (heads * dk,) and tau: sigmoid(decay_in + decay_bias)^(1 / tau).  -> fp32 (n, heads * dv)"""
     C.require_cuda(q, k, v, state, seqs, head_decay, decay_in, decay_bias)
-    if not (q.dtype == k.dtype == v.dtype) or state.dtype != torch.float32 or seqs.dtype != torch.int32 or not seqs.is_contiguous():
-        raise C.B200Error("linear_attn: q, k, v of one dtype, fp32 state, int32 seqs")
+    qk_f32 = q.dtype == torch.float32 and v.dtype != torch.float32 and head_decay is not None
+    if q.dtype != k.dtype or not (q.dtype == v.dtype or qk_f32) or state.dtype != torch.float32 or seqs.dtype != torch.int32 or not seqs.is_contiguous():
+        raise C.B200Error("linear_attn: q, k, v of one dtype (q and k also fp32 with fixed decays), fp32 state, int32 seqs")
     if (head_decay is None) == (decay_in is None):
         raise C.B200Error("linear_attn: either fixed decays per head or per-channel decays")
     if head_decay is not None and (head_decay.dtype != torch.float32 or head_decay.numel() != heads or not head_decay.is_contiguous()):
@@ -1023,7 +1084,7 @@ def linear_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.
                             q_scale=float(q_scale), decay_in=C.ptr(decay_in), ld_decay=0 if decay_in is None else decay_in.stride(0),
                             decay_bias=C.ptr(decay_bias), tau=float(tau), head_decay=C.ptr(head_decay), state=state.data_ptr(),
                             state_slot_stride=state.stride(0), out=out.data_ptr(), ldo=out.stride(0), seqs=seqs.data_ptr(), n_seqs=seqs.shape[0],
-                            rows=n, max_rows=int(max_rows), heads=heads, dk=dk, dv=dv, dtype=_code(q), workspace=C.ptr(ws),
+                            rows=n, max_rows=int(max_rows), heads=heads, dk=dk, dv=dv, dtype=_code(v), workspace=C.ptr(ws), qk_f32=int(qk_f32),
                             workspace_bytes=0 if ws is None else ws.numel() * ws.element_size())
     C.check(lib.b200_linear_attn(ctypes.byref(args), C.stream_ptr(q.device)), "linear_attn")
     return out
@@ -1037,14 +1098,25 @@ def linear_attn_tune(piece: int = 0) -> int:
 GATE_SILU, GATE_SIGMOID = 1, 2
 
 
-def gated_rms_heads(o: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, heads: int, dv: int, gate: int, eps: float) -> torch.Tensor:
-    """o fp32 (n, heads * dv), z (n, heads * dv) raw gate projection -> T (n, heads * dv): per-head RMS norm * weight * gate(z)."""
+def _out_rows(out: Optional[torch.Tensor], rows: int, cols: int, like: torch.Tensor, what: str) -> torch.Tensor:
+    """A destination (rows, cols) in `like`'s dtype: `out` itself, checked (it may be a column slice), or a new one."""
+    if out is None:
+        return torch.empty((rows, cols), dtype=like.dtype, device=like.device)
+    if tuple(out.shape) != (rows, cols) or out.dtype != like.dtype or out.stride(-1) != 1 or not out.is_cuda:
+        raise C.B200Error(f"{what}: the destination must be ({rows}, {cols}) in the operands' dtype with a unit inner stride")
+    return out
+
+
+def gated_rms_heads(o: torch.Tensor, z: torch.Tensor, weight: Optional[torch.Tensor], heads: int, dv: int, gate: int, eps: float, *, out_scale: float = 1.0,
+                    out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """o fp32 (n, heads * dv), z (n, heads * dv) raw gate projection -> T (n, heads * dv): per-head RMS norm * weight * gate(z) * out_scale,
+    in `out` when given (rows with unit inner stride); weight None: no weight."""
     C.require_cuda(o, z, weight)
-    if o.dtype != torch.float32 or o.stride(-1) != 1 or z.stride(-1) != 1 or z.dtype != weight.dtype:
+    if o.dtype != torch.float32 or o.stride(-1) != 1 or z.stride(-1) != 1 or (weight is not None and z.dtype != weight.dtype):
         raise C.B200Error("gated_rms_heads: o fp32, gate and weight in the model dtype")
-    out = torch.empty((o.shape[0], heads * dv), dtype=z.dtype, device=o.device)
-    C.check(C.load_core().b200_gated_rms_heads(o.data_ptr(), o.stride(0), z.data_ptr(), z.stride(0), weight.data_ptr(), out.data_ptr(), out.stride(0),
-                                               o.shape[0], heads, dv, gate, float(eps), _code(z), C.stream_ptr(o.device)), "gated_rms_heads")
+    out = _out_rows(out, o.shape[0], heads * dv, z, "gated_rms_heads")
+    C.check(C.load_core().b200_gated_rms_heads(o.data_ptr(), o.stride(0), z.data_ptr(), z.stride(0), C.ptr(weight), out.data_ptr(), out.stride(0),
+                                               o.shape[0], heads, dv, gate, float(eps), float(out_scale), _code(z), C.stream_ptr(o.device)), "gated_rms_heads")
     return out
 
 
@@ -1054,7 +1126,8 @@ WINDOW_PREFILL_MMA = True   # tests switch it off to run whole prompts with tens
 def window_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_ring: torch.Tensor, v_ring: torch.Tensor, sink: Optional[torch.Tensor],
                 seqs: torch.Tensor, row_seq: torch.Tensor, max_q_len: int, n_head: int, n_kv_head: int, dk: int, dv: int, window: int,
                 scale: float, from_start: bool = False, *, dist: Optional[Tuple[torch.Tensor, torch.Tensor]] = None,
-                gate: Optional[torch.Tensor] = None, gate_per_head: bool = False, keep: int = 0, softcap: float = 0.0) -> torch.Tensor:
+                gate: Optional[torch.Tensor] = None, gate_per_head: bool = False, keep: int = 0, softcap: float = 0.0,
+                out_scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Sliding-window attention with a sink over this step's k / v rows and the rings (slots, ring, G * dk | dv) of earlier
     positions; afterwards the step's rows enter the rings.  -> (n, n_head * dv).  from_start: every sequence of the step begins
     at position 0, so nothing is read from the rings -- bf16 prompts with 64- or 128-wide heads then run on the tensor-core tiles
@@ -1062,7 +1135,7 @@ def window_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_ring: torch
     projections of the rows (n, n_head) with gate_per_head, else (n, n_head * dv); the output is multiplied by their sigmoid.  keep: that
     many first positions stay visible to every later row (the rings then hold keep + ring rows per slot); softcap: scores become
     softcap * tanh(score / softcap) -- with either, bf16 prompts run on the tensor-core tiles for head sizes that are multiples of 8 up to
-    128, equal or not."""
+    128 (keys) and 256 (values).  The output is multiplied by out_scale, and goes to `out` when given (rows with unit inner stride)."""
     r1, r2 = dist if dist is not None else (None, None)
     C.require_cuda(q, k, v, k_ring, v_ring, sink, seqs, row_seq, r1, r2, gate)
     if dist is not None and not (r1.dtype == r2.dtype == q.dtype and r1.numel() == r2.numel() == n_head and r1.is_contiguous() and r2.is_contiguous()):
@@ -1076,10 +1149,10 @@ def window_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_ring: torch
     if q.stride(-1) != 1 or k.stride(-1) != 1 or v.stride(-1) != 1 or seqs.dtype != torch.int32 or not seqs.is_contiguous():
         raise C.B200Error("window_attn: unit inner strides, int32 seqs")
     ring = k_ring.shape[1] - keep
-    out = torch.empty((q.shape[0], n_head * dv), dtype=q.dtype, device=q.device)
+    out = _out_rows(out, q.shape[0], n_head * dv, q, "window_attn")
     lib, st = C.load_core(), C.stream_ptr(q.device)
     mma = from_start and max_q_len > 1 and WINDOW_PREFILL_MMA and q.dtype == torch.bfloat16
-    if (mma and keep == 0 and softcap == 0.0 and dk == dv and dk in (64, 128)
+    if (mma and keep == 0 and softcap == 0.0 and out_scale == 1.0 and dk == dv and dk in (64, 128)
             and not (q.stride(0) | k.stride(0) | v.stride(0)) & 7 and not (q.data_ptr() | k.data_ptr() | v.data_ptr() | seqs.data_ptr()) & 15):
         C.check(lib.b200_attn_prefill_window_ex(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), seqs.data_ptr(),
                                                 seqs.shape[0], max_q_len, out.data_ptr(), out.stride(0), n_head, n_kv_head, dk, float(scale), window,
@@ -1092,9 +1165,10 @@ def window_attn(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, k_ring: torch
                             ldq=q.stride(0), ldk=k.stride(0), ldv=v.stride(0), ldo=out.stride(0), k_ring=k_ring.data_ptr(), v_ring=v_ring.data_ptr(), sink=C.ptr(sink), seqs=seqs.data_ptr(),
                             n_seqs=seqs.shape[0], max_q_len=max_q_len, ring=ring, n_head=n_head, n_kv_head=n_kv_head, dk=dk, dv=dv, window=window,
                             scale=float(scale), dtype=_code(q), dist_r1=C.ptr(r1), dist_r2=C.ptr(r2), gate=C.ptr(gate), ldg=ldg, gate_mode=gate_mode,
-                            keep=keep, softcap=float(softcap))
-    if (mma and (keep > 0 or softcap > 0.0) and dist is None and scale > 0.0 and dk % 8 == 0 and dv % 8 == 0 and dk <= 128 and dv <= 128
-            and not (q.stride(0) | k.stride(0) | v.stride(0)) & 7 and not (q.data_ptr() | k.data_ptr() | v.data_ptr() | seqs.data_ptr()) & 15):
+                            keep=keep, softcap=float(softcap), out_scale=float(out_scale))
+    if (mma and (keep > 0 or softcap > 0.0) and dist is None and scale > 0.0 and dk % 8 == 0 and dv % 8 == 0 and dk <= 128 and dv <= 256
+            and not (q.stride(0) | k.stride(0) | v.stride(0)) & 7 and not (q.data_ptr() | k.data_ptr() | v.data_ptr() | seqs.data_ptr()) & 15
+            and not (out.stride(0) & 1 or out.data_ptr() & 3)):
         C.check(lib.b200_window_attn_tiles(ctypes.byref(args), st), "window_attn_tiles")
         C.check(lib.b200_ring_store_keep(k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), k_ring.data_ptr(), v_ring.data_ptr(), ring, keep,
                                          n_kv_head * dk, n_kv_head * dv, seqs.data_ptr(), row_seq.data_ptr(), q.shape[0], _code(q), st), "ring_store")
@@ -1140,9 +1214,10 @@ def rope_seg(inp: torch.Tensor, out: torch.Tensor, heads: int, dim: int, *, norm
              in_stride: Optional[int] = None, out_stride: Optional[int] = None, norm_all: bool = False) -> "C.HeadRopeSeg":
     """One group of `heads` heads of `dim` numbers for ``head_rope``: `inp` / `out` are 2-d views (rows, columns) whose first column
     is the group's first head; heads lie `in_stride` / `out_stride` (default dim) numbers apart.  freq: fp32 or fp64 (rot_dims / 2,).
-    norm_all: one norm over all heads of a row, norm_w of heads * dim numbers."""
-    if inp.stride(-1) != 1 or out.stride(-1) != 1 or inp.dtype != out.dtype:
-        raise C.B200Error("head_rope: rows of one dtype with unit inner stride")
+    norm_all: one norm over all heads of a row, norm_w of heads * dim numbers.  `out` may be fp32 for a 16-bit `inp`."""
+    f32 = out.dtype == torch.float32 and inp.dtype != torch.float32
+    if inp.stride(-1) != 1 or out.stride(-1) != 1 or not (inp.dtype == out.dtype or f32):
+        raise C.B200Error("head_rope: rows of one dtype (the destination also fp32) with unit inner stride")
     if freq is not None and (freq.dtype not in (torch.float32, torch.float64) or not freq.is_contiguous() or freq.numel() < rot_dims // 2):
         raise C.B200Error("head_rope: frequencies must be contiguous fp32 or fp64, one per rotated pair")
     if norm_all and (norm_w is None or norm_w.numel() != heads * dim or not norm_w.is_contiguous()):
@@ -1152,11 +1227,11 @@ def rope_seg(inp: torch.Tensor, out: torch.Tensor, heads: int, dim: int, *, norm
     return C.HeadRopeSeg(inp=inp.data_ptr(), out=out.data_ptr(), norm_w=C.ptr(norm_w), freq=C.ptr(freq) if rot_dims else None, out_rows=C.ptr(out_rows),
                          ld_in=inp.stride(-2), ld_out=out.stride(-2), heads=heads, dim=dim, in_stride=dim if in_stride is None else in_stride,
                          out_stride=dim if out_stride is None else out_stride, rot_off=rot_off, rot_dims=rot_dims, interleaved=int(interleaved),
-                         mag=float(mag), norm_all=int(norm_all), freq_f64=int(freq is not None and freq.dtype == torch.float64))
+                         mag=float(mag), norm_all=int(norm_all), freq_f64=int(freq is not None and freq.dtype == torch.float64), out_f32=int(f32))
 
 
 def head_rope(rows: int, row_pos: torch.Tensor, eps: float, *segs: "C.HeadRopeSeg", dtype: torch.dtype, device: torch.device) -> None:
-    """One launch over `rows` rows for up to three groups of heads built by ``rope_seg``: per head an optional weighted RMS norm, the
+    """One launch over `rows` rows for up to four groups of heads built by ``rope_seg``: per head an optional weighted RMS norm, the
     rotation of a run of its dimensions by the row's position, and the move to its destination (in place, dense, or cache rows)."""
     if row_pos.dtype != torch.int32 or not row_pos.is_contiguous():
         raise C.B200Error("head_rope: positions must be contiguous int32")

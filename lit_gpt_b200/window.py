@@ -113,9 +113,10 @@ class RingState(nn.Module):
 
 
 class GatedWindowAttention(nn.Module):
-    def __init__(self, width: int, spec: GatedWindowSpec, eps: float = 0.0, align: int = 1) -> None:
+    def __init__(self, width: int, spec: GatedWindowSpec, eps: float = 0.0, align: int = 1, projections: bool = True) -> None:
         """align: the fused projection gets zero rows at its end up to a multiple of `align` (rows of its result then start on 16-byte
-        boundaries whatever the number of heads)."""
+        boundaries whatever the number of heads).  projections=False: the input and output projections belong to whoever runs this
+        attention beside another mixer (``parallel``), through ``rope_segs`` and ``attend``."""
         super().__init__()
         self.spec, self.eps, self.width = spec, eps, width
         H, G, dk, dv = spec.heads, spec.kv_heads, spec.dim, spec.vdim
@@ -123,14 +124,14 @@ class GatedWindowAttention(nn.Module):
         self.cols = H * dk + G * dk + G * dv + self.gate_cols
         self.cols += -self.cols % align
         # fused projection: rows [0, H dk) queries, then G dk keys, G dv values, then the gate's rows (and padding)
-        self.w_in = nn.Parameter(torch.empty(self.cols, width), requires_grad=False)
-        self.b_in = nn.Parameter(torch.zeros(self.cols), requires_grad=False) if spec.bias else None
+        self.w_in = nn.Parameter(torch.empty(self.cols, width), requires_grad=False) if projections else None
+        self.b_in = nn.Parameter(torch.zeros(self.cols), requires_grad=False) if spec.bias and projections else None
         self.r1 = nn.Parameter(torch.zeros(H), requires_grad=False) if spec.distance else None
         self.r2 = nn.Parameter(torch.zeros(H), requires_grad=False) if spec.distance else None
         self.q_norm = nn.Parameter(torch.ones(H * dk), requires_grad=False) if spec.qk_norm else None
         self.k_norm = nn.Parameter(torch.ones(G * dk), requires_grad=False) if spec.qk_norm else None
         self.sink = nn.Parameter(torch.zeros(H), requires_grad=False) if spec.sink else None
-        self.w_o = nn.Parameter(torch.empty(width, H * dv), requires_grad=False)
+        self.w_o = nn.Parameter(torch.empty(width, H * dv), requires_grad=False) if projections else None
         self._freq_cache: dict = {}
 
     def freq(self, device: torch.device) -> Optional[torch.Tensor]:
@@ -148,6 +149,23 @@ class GatedWindowAttention(nn.Module):
         s = self.spec
         return RingState(slots, s.window, s.kv_heads * s.dim, s.kv_heads * s.vdim, device, dtype, keep=s.keep)
 
+    def rope_segs(self, q: torch.Tensor, k: torch.Tensor) -> list:
+        """Norms and rotations of the projected q and k, in place, as groups for ``K.head_rope`` (none where there is nothing to do)."""
+        s, fr = self.spec, self.freq(q.device)
+        if fr is None and not s.qk_norm:
+            return []
+        turn = dict(freq=fr, rot_dims=s.rot.dims, interleaved=s.rot.interleaved, mag=s.rot.magnitude) if fr is not None else {}
+        return [K.rope_seg(q, q, s.heads, s.dim, norm_w=self.q_norm, norm_all=s.qk_norm, **turn),
+                K.rope_seg(k, k, s.kv_heads, s.dim, norm_w=self.k_norm, norm_all=s.qk_norm, **turn)]
+
+    def attend(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: Optional[torch.Tensor], batch: RaggedBatch, state: RingState, *,
+               out_scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Attention over the step's rows and the rings, which the rows then enter -> (n, heads * vdim), times out_scale, in `out` if given."""
+        s = self.spec
+        return K.window_attn(q, k, v, state.k_ring, state.v_ring, self.sink, batch.seq_state, batch.row_seq, batch.max_q_len, s.heads, s.kv_heads, s.dim,
+                             s.vdim, s.window, s.scale, from_start=batch.identity_ctx, dist=(self.r1, self.r2) if s.distance else None, gate=gate,
+                             gate_per_head=s.gate == "head", keep=s.keep, softcap=s.softcap, out_scale=out_scale, out=out)
+
     def forward(self, h: torch.Tensor, batch: RaggedBatch, state: RingState) -> torch.Tensor:
         """h (n, width) in the matrix-product dtype -> (n, width)"""
         s, n = self.spec, h.shape[0]
@@ -156,12 +174,7 @@ class GatedWindowAttention(nn.Module):
         q, k, v = proj[:, : H * dk], proj[:, H * dk : (H + G) * dk], proj[:, (H + G) * dk : (H + G) * dk + G * dv]
         off = (H + G) * dk + G * dv
         gate = proj[:, off : off + self.gate_cols] if self.gate_cols else None
-        fr = self.freq(h.device)
-        if fr is not None or s.qk_norm:   # both norms and both rotations in place, one launch
-            turn = dict(freq=fr, rot_dims=s.rot.dims, interleaved=s.rot.interleaved, mag=s.rot.magnitude) if fr is not None else {}
-            K.head_rope(n, batch.row_pos, self.eps, K.rope_seg(q, q, H, dk, norm_w=self.q_norm, norm_all=s.qk_norm, **turn),
-                        K.rope_seg(k, k, G, dk, norm_w=self.k_norm, norm_all=s.qk_norm, **turn), dtype=h.dtype, device=h.device)
-        y = K.window_attn(q, k, v, state.k_ring, state.v_ring, self.sink, batch.seq_state, batch.row_seq, batch.max_q_len, H, G, dk, dv, s.window,
-                          s.scale, from_start=batch.identity_ctx, dist=(self.r1, self.r2) if s.distance else None, gate=gate,
-                          gate_per_head=s.gate == "head", keep=s.keep, softcap=s.softcap)
-        return F.linear(y, self.w_o)
+        segs = self.rope_segs(q, k)
+        if segs:   # both norms and both rotations in place, one launch
+            K.head_rope(n, batch.row_pos, self.eps, *segs, dtype=h.dtype, device=h.device)
+        return F.linear(self.attend(q, k, v, gate, batch, state), self.w_o)

@@ -280,7 +280,9 @@ class RotarySpec:
     """Rotary positions on the first `dims` dimensions of a head, frequency base^(-2i / dims) for pair i; pairs are (2i, 2i + 1)
     when `interleaved`, else (i, i + dims / 2).  With `factor` set the frequencies are blended towards f / factor over a ramp
     between the dimensions whose wavelength fits `fast` and `slow` times into `original` positions (YaRN), and cos / sin are
-    scaled by 0.1 ln(factor) + 1."""
+    scaled by 0.1 ln(factor) + 1.  With `high` set as well the blend goes by the wavelength itself (Llama 3.1): a pair that turns
+    t = original / wavelength times keeps f for t > high, gets f / factor for t < low, and in between s f + (1 - s) f / factor with
+    s = (t - low) / (high - low); cos / sin unscaled."""
 
     dims: int
     base: float
@@ -289,13 +291,15 @@ class RotarySpec:
     fast: float = 32.0
     slow: float = 1.0
     interleaved: bool = True
+    low: float = 0.0
+    high: float = 0.0
 
     @classmethod
     def from_dict(cls, rot: Dict[str, Any], interleaved: bool = True) -> "RotarySpec":
         sc = rot.get("scaling") or {}
         return cls(dims=int(rot["dims"]), base=float(rot["base"]), factor=float(sc["factor"]) if sc else None,
                    original=float(sc.get("original", 0.0)), fast=float(sc.get("fast", 32.0)), slow=float(sc.get("slow", 1.0)),
-                   interleaved=interleaved)
+                   interleaved=interleaved, low=float(sc.get("low", 0.0)), high=float(sc.get("high", 0.0)))
 
     def frequencies(self) -> List[float]:
         """Angular frequency of every pair, as Python floats (double precision)."""
@@ -305,6 +309,17 @@ class RotarySpec:
         f = [self.base ** (-2.0 * i / self.dims) for i in range(half)]
         if self.factor is None:
             return f
+        if self.high > 0.0:
+            def blend(fi: float) -> float:
+                turns = self.original * fi / (2.0 * math.pi)
+                if turns > self.high:
+                    return fi
+                if turns < self.low:
+                    return fi / self.factor
+                s = (turns - self.low) / (self.high - self.low) if self.high > self.low else 0.0
+                return (1.0 - s) * fi / self.factor + s * fi
+
+            return [blend(fi) for fi in f]
 
         def pair_of(turns: float) -> float:   # the (fractional) pair index whose wavelength makes `turns` turns over `original`
             return self.dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
@@ -321,7 +336,7 @@ class RotarySpec:
     def magnitude(self) -> float:
         import math
 
-        return 1.0 if self.factor is None else 0.1 * math.log(self.factor) + 1.0
+        return 1.0 if self.factor is None or self.high > 0.0 else 0.1 * math.log(self.factor) + 1.0
 
 
 @dataclass
@@ -839,12 +854,132 @@ class VotavikConfig:
             return cls.from_dict(json.load(fp))
 
 
+@dataclass
+class RetentionSpec:
+    """Retention: linear attention S <- decay_h S + k v^T, o = S^T q with one fixed decay per head; rotary positions (half-split pairs) on
+    q and k, k times dim^-1/2; every head's o over its own root mean square (no weight), then a silu output gate."""
+
+    heads: int
+    dim: int
+    vdim: int
+    decay: List[float] = field(default_factory=list)
+    rot: Optional[RotarySpec] = None
+
+
+@dataclass
+class WindowRetentionSpec:
+    """Sliding-window attention (left) and retention (right) on the same input: left_scale * left + right_scale * right."""
+
+    left: GatedWindowSpec
+    right: RetentionSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+
+@dataclass
+class SharedMoESpec:
+    """Experts W_down (silu(W_gate h) * (W_up h)) chosen by the largest router logits, weighted by a softmax among those `top` logits;
+    optionally a shared expert of the same form (its own ff) for every token, times the sigmoid of one projected number per token."""
+
+    experts: int
+    top: int
+    ff: int
+    shared_ff: int = 0             # 0: no shared expert
+
+
+@dataclass
+class FoviraxLayerSpec:
+    type: str                      # "parallel"
+    mixer: WindowRetentionSpec
+    mlp: Optional[SharedMoESpec] = None
+
+
+@dataclass
+class FoviraxConfig:
+    """Fovirax: pre-normed blocks (RMS norms whose weights are stored around zero) over an fp32 residual stream, every sublayer's result
+    scaled per channel and by one constant.  Mixer: sliding-window attention with capped scores and retention side by side; feed-forward:
+    sparse experts with a gated shared one, or none.  Layers loop_start .. loop_stop - 1 run loop_times times with the same weights, each
+    pass with its own state."""
+
+    name: str = "Fovirax"
+    vocab_size: int = 0
+    n_embd: int = 0
+    norm_eps: float = 1e-5
+    residual_mult: float = 1.0
+    layers: List[FoviraxLayerSpec] = field(default_factory=list)
+    loop_start: int = 0
+    loop_stop: int = 0
+    loop_times: int = 1
+    block_size: int = 1 << 30      # constant-size state, no position table: positions are bounded by int32 only
+
+    def __post_init__(self) -> None:
+        self.padded_vocab_size = self.vocab_size
+        self.n_layer = len(self.layers)
+        if self.loop_times < 1 or not 0 <= self.loop_start <= self.loop_stop <= self.n_layer:
+            raise ValueError(f"loop {self.loop_start}..{self.loop_stop} x {self.loop_times} does not fit {self.n_layer} layers")
+        for i, layer in enumerate(self.layers):
+            if layer.type != "parallel":
+                raise ValueError(f"layer {i}: unknown mixer type {layer.type!r}")
+            lf, rt, e = layer.mixer.left, layer.mixer.right, layer.mlp
+            if lf.heads < 1 or lf.kv_heads < 1 or lf.heads % lf.kv_heads or lf.window < 1 or lf.dim < 1 or lf.vdim < 1 or lf.softcap < 0:
+                raise ValueError(f"layer {i}: bad attention shape")
+            if rt.heads < 1 or rt.dim < 1 or rt.vdim < 1:
+                raise ValueError(f"layer {i}: bad retention shape")
+            if len(rt.decay) != rt.heads or not all(0.0 <= g <= 1.0 for g in rt.decay):
+                raise ValueError(f"layer {i}: one decay in [0, 1] per head")
+            for m in (lf, rt):
+                if m.rot is not None and (m.rot.dims % 2 or m.rot.dims > m.dim):
+                    raise ValueError(f"layer {i}: rotary dimensions must be even and at most the head size")
+            if e is not None and (not 0 < e.top <= e.experts or e.ff < 1 or e.shared_ff < 0):
+                raise ValueError(f"layer {i}: bad expert shape (top {e.top} of {e.experts})")
+
+    def schedule(self) -> List[Tuple[int, int]]:
+        """The layer runs in order: (layer index, state index).  Every run has a state of its own."""
+        order = list(range(self.loop_start)) + list(range(self.loop_start, self.loop_stop)) * self.loop_times + list(range(self.loop_stop, self.n_layer))
+        return [(i, n) for n, i in enumerate(order)]
+
+    @classmethod
+    def from_dict(cls, js: Dict[str, Any]) -> "FoviraxConfig":
+        def rotary(mx: Dict[str, Any]) -> Optional[RotarySpec]:
+            rot = mx.get("rot")
+            return RotarySpec.from_dict(rot, interleaved=False) if rot and int(rot["dims"]) > 0 else None
+
+        layers = []
+        for i, entry in enumerate(js["layers"]):
+            if entry["type"] != "parallel":
+                raise ValueError(f"layer {i}: unknown mixer type {entry['type']!r}")
+            mx = entry["mixer"]
+            lf, rt = mx["left"], mx["right"]
+            left = GatedWindowSpec(heads=int(lf["heads"]), kv_heads=int(lf.get("kv_heads", lf["heads"])), dim=int(lf["dim"]), vdim=int(lf.get("vdim", lf["dim"])),
+                                   window=int(lf["mask"]["size"]), scale=float(lf["scale"]), rot=rotary(lf), gate=None, softcap=float(lf.get("softcap") or 0.0))
+            right = RetentionSpec(heads=int(rt["heads"]), dim=int(rt["dim"]), vdim=int(rt.get("vdim", rt["dim"])), decay=[float(g) for g in rt["decay"]],
+                                  rot=rotary(rt))
+            mixer = WindowRetentionSpec(left=left, right=right, left_scale=float(mx.get("left_scale", 1.0)), right_scale=float(mx.get("right_scale", 1.0)))
+            mlp, ml = None, entry.get("mlp")
+            if ml is not None:
+                if ml.get("kind", "moe") != "moe":
+                    raise ValueError(f"layer {i}: unknown feed-forward kind {ml.get('kind')!r}")
+                mlp = SharedMoESpec(experts=int(ml["router"]["experts"]), top=int(ml["router"]["top"]), ff=int(ml["expert"]["ff"]),
+                                    shared_ff=int((ml.get("shared") or {}).get("ff", 0)))
+            layers.append(FoviraxLayerSpec(type=entry["type"], mixer=mixer, mlp=mlp))
+        loop = js.get("loop") or {}
+        return cls(name=js.get("architecture", "Fovirax"), vocab_size=int(js["vocab"]), n_embd=int(js["width"]), norm_eps=float(js["norm"]["eps"]),
+                   residual_mult=float(js.get("residual_mult", 1.0)), layers=layers, loop_start=int(loop.get("start", 0)),
+                   loop_stop=int(loop.get("stop", loop.get("start", 0))), loop_times=int(loop.get("times", 1)))
+
+    @classmethod
+    def from_json(cls, path: Union[str, Path]) -> "FoviraxConfig":
+        with open(path, encoding="utf-8") as fp:
+            return cls.from_dict(json.load(fp))
+
+
 # "architecture" value of config.json -> (configuration class, "module:class" of the model)
 architectures: Dict[str, Any] = {"Pomipel": (PomipelConfig, "lit_gpt_b200.pomipel:Pomipel"),
                                  "Lefalix": (LefalixConfig, "lit_gpt_b200.lefalix:Lefalix"),
                                  "Fizadra": (FizadraConfig, "lit_gpt_b200.fizadra:Fizadra"),
                                  "Nulezen": (NulezenConfig, "lit_gpt_b200.nulezen:Nulezen"),
-                                 "Votavik": (VotavikConfig, "lit_gpt_b200.votavik:Votavik")}
+                                 "Votavik": (VotavikConfig, "lit_gpt_b200.votavik:Votavik"),
+                                 "Fovirax": (FoviraxConfig, "lit_gpt_b200.fovirax:Fovirax")}
 
 
 def load_config(checkpoint_dir: Union[str, Path], **kwargs: Any) -> Any:

@@ -32,17 +32,9 @@ from . import kernels as K
 from .config import DenseMLPSpec, GatedMoESpec, LefalixConfig, LefalixLayerSpec
 from .delta import GatedDeltaRule
 from .moe import DenseMLP, GatedSparseExperts
+from .parallel import ParallelState
 from .ragged import RaggedBatch, StateServed
 from .window import WindowAttention
-
-
-class ParallelState(nn.Module):
-    def __init__(self, left: nn.Module, right: nn.Module) -> None:
-        super().__init__()
-        self.left, self.right = left, right
-
-    def tensors(self) -> List[torch.Tensor]:
-        return self.left.tensors() + self.right.tensors()
 
 
 class ParallelMixer(nn.Module):

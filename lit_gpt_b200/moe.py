@@ -14,14 +14,21 @@ and up rows stacked into one (experts, 2 ff, width) tensor so that both are one 
 ``ClampedSparseExperts``: the router adds a bias to its logits, takes the `top` largest and weights them by a softmax among
 those few; experts are gated with clamped branches, W_down (g sigmoid(alpha g) (u + 1)), g = min(W_gate x, limit), u = clamp(W_up x,
 -limit, limit); ``ClampedGLU`` is one such expert for every token (a shared expert).
+
+``SharedSparseExperts``: the `top` largest logits weighted by a softmax among them, plain gated experts W_down (silu(W_gate x) * (W_up x)),
+and a shared expert of that form times the sigmoid of one projected number per token.  The router's rows and that number's row are
+one weight: few tokens run them in the routing kernel, many as one matrix product with fp32 logits.  ``terms`` hands the parts of the
+result to the residual kernel, which weights and sums them (``K.gated_residual``).
 """
 from __future__ import annotations
+
+from typing import Dict
 
 import torch
 import torch.nn as nn
 
 from . import kernels as K
-from .config import ClampedMoESpec, GatedMoESpec, MoESpec
+from .config import ClampedMoESpec, GatedMoESpec, MoESpec, SharedMoESpec
 
 
 VENDOR_GROUPED_GEMM = True   # tests switch it off to run the library's own grouped kernel on the same input
@@ -122,6 +129,53 @@ class ClampedSparseExperts(nn.Module):
         both = torch._grouped_mm(K.gather_rows(x, plan.slot_token), self.w_up.transpose(1, 2), offs=ends)
         y = torch._grouped_mm(K.glu_clamped(both, sp.limit, sp.alpha), self.w_down.transpose(1, 2), offs=ends)
         return K.moe_combine(y, plan, weights)
+
+
+class SharedSparseExperts(nn.Module):
+    ROUTE_MM_MIN_ROWS = 32    # from this many tokens on the router's logits are one matrix product
+
+    def __init__(self, width: int, spec: SharedMoESpec) -> None:
+        super().__init__()
+        self.spec = spec
+        E, ff, ffs = spec.experts, spec.ff, spec.shared_ff
+        route_rows = E + (1 if ffs else 0)
+        # the router's rows, then the row of the shared expert's gate, then zero rows up to a multiple of 8
+        self.w_route = nn.Parameter(torch.empty(route_rows + -route_rows % 8, width), requires_grad=False)
+        self.w_up = nn.Parameter(torch.empty(E, 2 * ff, width), requires_grad=False)   # per expert: ff gate rows, then ff up rows
+        self.w_down = nn.Parameter(torch.empty(E, width, ff), requires_grad=False)
+        self.shared_up = nn.Parameter(torch.empty(2 * ffs, width), requires_grad=False) if ffs else None
+        self.shared_down = nn.Parameter(torch.empty(width, ffs), requires_grad=False) if ffs else None
+
+    def route(self, x: torch.Tensor):
+        """-> expert ids int32 (n, top), their weights fp32 (n, top), the shared expert's gate fp32 (n,) or None"""
+        sp, shared = self.spec, self.shared_up is not None
+        if x.shape[0] >= self.ROUTE_MM_MIN_ROWS and sp.top <= 32 and sp.experts <= 3072:
+            res = K.moe_route_logits(K.mm_f32(x, self.w_route), sp.experts, sp.top, gate=shared)
+        else:
+            res = K.moe_route(x, self.w_route[: sp.experts], None, sp.top, 1, 1, topk_softmax=True, gate_w=self.w_route[sp.experts] if shared else None)
+        return res if shared else (*res, None)
+
+    def terms(self, x: torch.Tensor) -> Dict[str, torch.Tensor]:
+        """The parts of the feed-forward's result as keyword arguments of ``K.gated_residual``."""
+        sp, (n, d) = self.spec, x.shape
+        ids, weights, gate = self.route(x)
+        few = n * sp.top <= K.MOE_GEMV_MAX_PAIRS
+        if few and self.shared_up is not None:
+            y0, y1 = K.moe_experts_shared(x, ids, weights, self.w_up, self.w_down, self.shared_up, self.shared_down)
+            return dict(y0=y0, y1=y1, gate=gate)
+        res: Dict[str, torch.Tensor] = {}
+        if few or x.dtype != torch.bfloat16 or d % 8 or sp.ff % 8 or not VENDOR_GROUPED_GEMM or not hasattr(torch, "_grouped_mm"):
+            res["y0"] = K.moe_experts(x, ids, weights, self.w_up, self.w_down, gated=True)
+        else:
+            plan = K.moe_plan(ids, sp.experts)
+            ends = plan.expert_off[1:]
+            both = torch._grouped_mm(K.gather_rows(x, plan.slot_token), self.w_up.transpose(1, 2), offs=ends)
+            res["y0"] = torch._grouped_mm(K.glu(both, K.ACT_SILU), self.w_down.transpose(1, 2), offs=ends)
+            res["slot_of"], res["wts"] = plan.slot_of, weights
+        if self.shared_up is not None:
+            hidden = K.glu(torch.nn.functional.linear(x, self.shared_up), K.ACT_SILU)
+            res["y1"], res["gate"] = torch.nn.functional.linear(hidden, self.shared_down), gate
+        return res
 
 
 class DenseMLP(nn.Module):

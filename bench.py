@@ -1265,6 +1265,157 @@ def run_votavik_compare(args) -> None:
                       "gpu_launches": int(K.launch_count() - launches0), "sizes": out}), flush=True)
 
 
+# ---------------------------------------------------------------------------------------------------------
+# --compare fovirax: the Fovirax design beside the closest existing model (Lefalix: the other design with windowed attention and a recurrent
+# mixer side by side and sparse gated experts) at equal width, heads, head size, window, layers and weights used per token (one chosen
+# expert less, a shared one of the same size instead); single kernels also beside Votavik's capped attention and linear attention.
+# ---------------------------------------------------------------------------------------------------------
+def run_fovirax_compare(args) -> None:
+    from lit_gpt_b200 import kernels as K
+    from lit_gpt_b200.config import (DeltaMixerSpec, FoviraxConfig, FoviraxLayerSpec, GatedMoESpec, GatedWindowSpec, LefalixConfig, LefalixLayerSpec,
+                                     ParallelMixerSpec, RetentionSpec, RotarySpec, SharedMoESpec, WindowMixerSpec, WindowRetentionSpec)
+    from lit_gpt_b200.fovirax import Fovirax
+    from lit_gpt_b200.lefalix import Lefalix
+    from lit_gpt_b200.ragged import state_batch
+
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    peaks, peak_source = measured_peaks()
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    flush = torch.zeros(256 << 20, dtype=torch.uint8, device=dev)
+    vocab, T, cap, layers = 32000, args.prompt, 30.0, 4
+    iters = max(3, min(args.steps, 20))
+    launches0 = K.launch_count()
+    bf = torch.bfloat16
+    out = {}
+    for name in (args.sizes.split(",") if args.sizes else LEFALIX_SIZES):
+        d, H, G, hs, W, _, E, top, ff, _ = LEFALIX_SIZES[name]
+        Hr = H // 2
+        rot = RotarySpec(dims=hs, base=1e6, interleaved=False, factor=4.0, original=4096.0, low=1.0, high=4.0)
+        decay = [1 - 2.0 ** -(5 + j % 8) for j in range(Hr)]
+        fov_layer = lambda: FoviraxLayerSpec("parallel", WindowRetentionSpec(GatedWindowSpec(H, G, hs, hs, W, hs ** -0.5, rot=rot, gate=None, softcap=cap),   # noqa: E731
+                                                                             RetentionSpec(Hr, hs, hs, decay, RotarySpec(dims=hs, base=1e4, interleaved=False)), 0.7, 0.9),
+                                             SharedMoESpec(E, top - 1, ff, ff))
+        fov = Fovirax(FoviraxConfig(vocab_size=vocab, n_embd=d, residual_mult=0.5, layers=[fov_layer() for _ in range(layers)])).to(dev).to(bf).eval()
+        fov.reset_parameters()
+        fov.max_seq_length = T + 64
+        lrot = RotarySpec(dims=hs, base=1e6, factor=4.0, original=4096.0, fast=32.0, slow=1.0)
+        lef_layer = lambda: LefalixLayerSpec("parallel", ParallelMixerSpec(WindowMixerSpec(H, G, hs, hs, 4, W, hs ** -0.5, lrot), DeltaMixerSpec(Hr, Hr // 2, hs, hs, 4)),   # noqa: E731
+                                             GatedMoESpec(E, top, ff))
+        lef = Lefalix(LefalixConfig(vocab_size=vocab, n_embd=d, layers=[lef_layer() for _ in range(layers)])).to(dev).to(bf).eval()
+        lef.reset_parameters()
+        lef.max_seq_length = T + 64
+        res = {}
+        with torch.inference_mode():
+            for label, model in (("fovirax", fov), ("lefalix", lef)):
+                for B in (1, 8):
+                    model.set_kv_cache(batch_size=B)
+                    idx = torch.randint(0, vocab, (B, T), device=dev)
+                    pos = torch.arange(T, device=dev)
+                    if B == 1:
+                        ms = _timed(lambda: model(idx, pos), iters, flush)
+                        res[f"{label}_prefill_tok_s"] = round(T / ms * 1e3)
+                    else:
+                        model(idx, pos)
+                    tok, p1 = idx[:, :1].contiguous(), torch.tensor([T], device=dev)
+                    step, graphed = _graphed(lambda: model(tok, p1))
+                    ms = _timed(step, iters, flush)
+                    res[f"{label}_decode_b{B}_tok_s"] = round(B / ms * 1e3)
+                    res[f"{label}_decode_b{B}_graphed"] = graphed
+                    del step
+                model.clear_kv_cache()
+            kern = {}
+
+            def put(key, fn, *, nbytes=None, flops=None, n=iters):
+                ms = _timed(fn, n, flush)
+                kern[key] = {"ms": ms}
+                if flops is not None:
+                    kern[key]["frac_of_measured_bf16"] = flops / (ms * 1e-3) / tf
+                if nbytes is not None:
+                    kern[key]["frac_of_measured_hbm"] = nbytes / (ms * 1e-3) / hbm
+
+            B = 8
+            batch, _ = state_batch([(0, 0, T)], dev, positions=True)
+            bd, _ = state_batch([(b, T, 1) for b in range(B)], dev, positions=True)
+            # windowed attention; values as wide as keys (all three designs) and twice as wide (this one)
+            pairs, keep = sum(min(i + 1, W) for i in range(T)), 4
+            q, kk = torch.randn(T, H * hs, device=dev, dtype=bf), torch.randn(T, G * hs, device=dev, dtype=bf)
+            sink, gate_h = torch.zeros(H, device=dev, dtype=bf), torch.randn(T, H, device=dev, dtype=bf)
+            for label, dv, kp, sc, kw in (("fovirax_cap", hs, 0, cap, {}), ("fovirax_cap_values_twice_as_wide", 2 * hs, 0, cap, {}),
+                                          ("votavik_kept_cap_sink_gate_per_head", hs, keep, cap, dict(sink=sink, gate=gate_h, gate_per_head=True)),
+                                          ("lefalix_sink", hs, 0, 0.0, dict(sink=sink))):
+                vv, rings = torch.randn(T, G * dv, device=dev, dtype=bf), [torch.randn(B, W + kp, G * m, device=dev, dtype=bf) for m in (hs, dv)]
+
+                def win(b, rows, n_rows):
+                    cut = {nm: (t[:rows] if nm == "gate" else t) for nm, t in kw.items()}
+                    return K.window_attn(q[:rows], kk[:rows], vv[:rows], *rings, cut.pop("sink", None), b.seq_state, b.row_seq, n_rows, H, G, hs, dv, W, hs ** -0.5,
+                                         from_start=n_rows > 1, keep=kp, softcap=sc, **cut)
+
+                put(f"prefill_attention_{label}", lambda: win(batch, T, T), flops=2.0 * H * (hs + dv) * pairs)
+                put(f"decode_attention_{label}", lambda: win(bd, B, 1), nbytes=1.0 * B * G * (W + kp) * (hs + dv) * 2)
+            # rotation: four groups (two into fp32) beside Votavik's norm and rotation of two groups in place
+            mx = fov.blocks[0].mixer
+            proj = torch.randn(T, mx.w_in.shape[0], device=dev, dtype=bf)
+            lq, lk, lv, rq, rk, rv, rg = (proj[:, at : at + rows] for at, (_, rows) in zip(mx.offsets, mx.rows))
+            tq, tk, segs = mx.right.turned(rq, rk)
+            segs = mx.left.rope_segs(lq, lk) + segs
+            put("rotation_four_groups_fovirax", lambda: K.head_rope(T, batch.row_pos, 0.0, *segs, dtype=bf, device=dev), nbytes=T * hs * ((H + G) * 4.0 + 2 * Hr * 6.0))
+            w_q, w_k = torch.ones(H * hs, device=dev, dtype=bf), torch.ones(G * hs, device=dev, dtype=bf)
+            turn = dict(freq=mx.left.freq(dev), rot_dims=hs, interleaved=False)
+            put("norm_over_heads_rotation_votavik", lambda: K.head_rope(T, batch.row_pos, 1e-5, K.rope_seg(lq, lq, H, hs, norm_w=w_q, norm_all=True, **turn),
+                                                                        K.rope_seg(lk, lk, G, hs, norm_w=w_k, norm_all=True, **turn), dtype=bf, device=dev),
+                nbytes=T * (H + G) * hs * 4.0)
+            # recurrences
+            hd, st = mx.right.constants(dev)[0], torch.zeros(B, Hr * hs * hs, device=dev)
+            put("prompt_retention_fovirax", lambda: K.linear_attn(tq, tk, rv, st, batch.seq_state, T, Hr, hs, hs, q_scale=hs ** -0.5, head_decay=hd),
+                nbytes=T * Hr * hs * (8 + 2 + 4.0))
+            put("prompt_linear_attention_per_head_votavik", lambda: K.linear_attn(rq, rk, rv, st, batch.seq_state, T, Hr, hs, hs, silu=True, head_decay=hd),
+                nbytes=T * Hr * hs * (4 + 2 + 4.0))
+            Gl = max(1, Hr // 2)
+            qf, kf = (torch.nn.functional.normalize(torch.randn(T, Gl, hs, device=dev), dim=-1).view(T, -1) for _ in range(2))
+            vf, bt, dh = torch.randn(T, Hr * hs, device=dev), torch.randn(T, Hr, device=dev, dtype=bf), torch.randn(T, Hr, device=dev, dtype=bf)
+            zero, std = torch.zeros(Hr, device=dev, dtype=bf), torch.zeros(B, Hr * K.delta_rule_state_floats(hs, hs), device=dev)
+            put("prompt_delta_rule_lefalix", lambda: K.delta_rule(qf, kf, vf, bt, dh, zero, zero, std, batch.seq_state, Hr, Gl, hs, hs, False, max_rows=T),
+                nbytes=T * (2 * Gl + 2 * Hr) * hs * 4.0)
+            states = 2.0 * B * Hr * hs * hs * 4
+            put("decode_retention_fovirax", lambda: K.linear_attn(tq[:B], tk[:B], rv[:B], st, bd.seq_state, 1, Hr, hs, hs, q_scale=hs ** -0.5, head_decay=hd), nbytes=states)
+            put("decode_linear_attention_per_head_votavik", lambda: K.linear_attn(rq[:B], rk[:B], rv[:B], st, bd.seq_state, 1, Hr, hs, hs, silu=True, head_decay=hd),
+                nbytes=states)
+            put("decode_delta_rule_lefalix", lambda: K.delta_rule(qf[:B], kf[:B], vf[:B], bt[:B], dh[:B], zero, zero, std, bd.seq_state, Hr, Gl, hs, hs, False, max_rows=1),
+                nbytes=states)
+            o, w1 = torch.randn(T, Hr * hs, device=dev), torch.ones(hs, device=dev, dtype=bf)
+            put("gated_norm_without_weight_fovirax", lambda: K.gated_rms_heads(o, rg, None, Hr, hs, K.GATE_SILU, 1e-5, out_scale=0.9), nbytes=T * Hr * hs * 8.0)
+            put("gated_norm_votavik_and_lefalix", lambda: K.gated_rms_heads(o, rg, w1, Hr, hs, K.GATE_SILU, 1e-5), nbytes=T * Hr * hs * 8.0)
+            # residual kernels
+            x, xs, act = torch.randn(T, d, device=dev, dtype=bf), torch.randn(T, d, device=dev), torch.empty(T, d, device=dev, dtype=bf)
+            fb, lb = fov.blocks[0], lef.blocks[0]
+            put("residual_mixer_fovirax", lambda: K.gated_residual(xs, x, 1e-5, scale=fb.ls1, mult=0.5, norm_w=fb.norm_2, plus_one=True, act=act), nbytes=T * d * 12.0)
+            terms = fb.mlp.terms(x)
+            put("residual_experts_fovirax", lambda: K.gated_residual(xs, eps=1e-5, scale=fb.ls2, mult=0.5, norm_w=fb.norm_1, plus_one=True, act=act, **terms),
+                nbytes=T * d * (12.0 + 2 * (top - 1)))
+            put("residual_lefalix", lambda: K.sandwich_residual(xs, x, lb.norm_1b, 1e-5, pre_w=lb.norm_2, act=act), nbytes=T * d * 12.0)
+            # experts: prompts, and a few tokens (the weights of the experts in use are what has to move)
+            put("route_prompt_fovirax", lambda: fb.mlp.route(x), nbytes=T * d * 2.0)
+            put("route_prompt_lefalix", lambda: lb.mlp.router(x), nbytes=T * d * 2.0)
+            put("experts_prompt_fovirax", lambda: fb.mlp.terms(x), flops=6.0 * T * top * ff * d)
+            put("experts_prompt_lefalix", lambda: lb.mlp(x), flops=6.0 * T * top * ff * d)
+            for n in (1, B):
+                used = fb.mlp.route(x[:n])[0].unique().numel() + 1
+                put(f"experts_{n}_token_fovirax", lambda: fb.mlp.terms(x[:n]), nbytes=used * 6.0 * ff * d)
+                put(f"route_{n}_token_fovirax", lambda: fb.mlp.route(x[:n]), nbytes=2.0 * (E + 1) * d)
+                used = lb.mlp.router(x[:n])[0].unique().numel()
+                put(f"experts_{n}_token_lefalix", lambda: lb.mlp(x[:n]), nbytes=used * 6.0 * ff * d)
+                put(f"route_{n}_token_lefalix", lambda: lb.mlp.router(x[:n]), nbytes=2.0 * E * d)
+            res["kernels"] = {k_: {a: (round(b_, 4) if isinstance(b_, float) else b_) for a, b_ in v_.items()} for k_, v_ in kern.items()}
+        out[name] = res
+        del fov, lef, fb, lb, mx, terms
+        torch.cuda.empty_cache()
+    print(json.dumps({"compare": "fovirax", "layers": layers, "prompt": T, "context": T, "dtype": "bf16", "data": "synthetic, random weights",
+                      "l2": "flushed between timed calls", "peaks": {"hbm_gbs": peaks["hbm_gbs"], "bf16_tflops": peaks["bf16_tflops"],
+                                                                       "source": peak_source},
+                      "gpu_launches": int(K.launch_count() - launches0), "sizes": out}), flush=True)
+
+
 def main() -> None:
     # stdout carries exactly one JSON line: NCCL's own banner / debug lines (when the box sets NCCL_DEBUG) go to stderr
     os.environ.setdefault("NCCL_DEBUG_FILE", "/dev/stderr")
@@ -1278,11 +1429,14 @@ def main() -> None:
     ap.add_argument("--workload", choices=sorted(WORKLOADS), default="llama2-7b-nf4-bs1")
     ap.add_argument("--layers", type=int, default=None, help="debug only: build fewer blocks (invalidates the number)")
     ap.add_argument("--no-cpu-baseline", action="store_true")
-    ap.add_argument("--compare", choices=["pomipel", "lefalix", "fizadra", "nulezen", "votavik"], default=None,
+    ap.add_argument("--compare", choices=["pomipel", "lefalix", "fizadra", "nulezen", "votavik", "fovirax"], default=None,
                     help="instead of the default workload: prefill / decode throughput of that design beside the closest existing model")
     ap.add_argument("--sizes", default=None, help=f"--compare: comma-separated subset of {sorted(ARCH_SIZES)} (the same names for both designs)")
     ap.add_argument("--prompt", type=int, default=2048, help="--compare: prompt and context length")
     args = ap.parse_args()
+    if args.compare == "fovirax":
+        run_fovirax_compare(args)
+        return
     if args.compare == "votavik":
         run_votavik_compare(args)
         return

@@ -277,26 +277,29 @@ struct SharedExpert {
   int ff, tokens;
 };
 
-// dot products of one or two weight rows with up to kShTok token rows (row pitch n); every lane gets the sums
-template <typename T, int NW>
-__device__ __forceinline__ void shared_dots(const T* __restrict__ w, int64_t w_pitch, const T* __restrict__ x, int n, int nt, int lane, float (&acc)[NW][kShTok]) {
+// dot products of NW weight rows with NT token rows (row pitch n), of which nt <= NT are there (the last one stands in for the others, so
+// that all loads of a pass can be in flight together); every lane gets the sums
+template <typename T, int NW, int NT>
+__device__ __forceinline__ void shared_dots_of(const T* __restrict__ w, int64_t w_pitch, const T* __restrict__ x, int n, int nt, int lane, float (&acc)[NW][kShTok]) {
 #pragma unroll
   for (int r = 0; r < NW; ++r)
 #pragma unroll
-    for (int t = 0; t < kShTok; ++t) acc[r][t] = 0.f;
+    for (int t = 0; t < NT; ++t) acc[r][t] = 0.f;
+  const T* xt[NT];
+#pragma unroll
+  for (int t = 0; t < NT; ++t) xt[t] = x + (int64_t)min(t, nt - 1) * n;
   bool vec = vec8_ok(n, w, x);
   if (NW > 1) vec = vec && vec8_ok(w_pitch, w);
   if (vec) {
-#pragma unroll 2
+#pragma unroll (NT > 2 ? 1 : 4)
     for (int i = lane * 8; i < n; i += 256) {
       float a[NW][8];
 #pragma unroll
       for (int r = 0; r < NW; ++r) load8(w + r * w_pitch + i, a[r]);
 #pragma unroll
-      for (int t = 0; t < kShTok; ++t) {
-        if (t >= nt) break;
+      for (int t = 0; t < NT; ++t) {
         float v[8];
-        load8(x + (int64_t)t * n + i, v);
+        load8(xt[t] + i, v);
 #pragma unroll
         for (int r = 0; r < NW; ++r)
 #pragma unroll
@@ -309,20 +312,25 @@ __device__ __forceinline__ void shared_dots(const T* __restrict__ w, int64_t w_p
 #pragma unroll
       for (int r = 0; r < NW; ++r) a[r] = load_as_float(w, r * w_pitch + i);
 #pragma unroll
-      for (int t = 0; t < kShTok; ++t) {
-        if (t >= nt) break;
-        const float v = load_as_float(x, (int64_t)t * n + i);
+      for (int t = 0; t < NT; ++t) {
+        const float v = load_as_float(xt[t], i);
 #pragma unroll
         for (int r = 0; r < NW; ++r) acc[r][t] = fmaf(a[r], v, acc[r][t]);
       }
     }
   }
 #pragma unroll
-  for (int t = 0; t < kShTok; ++t) {
-    if (t >= nt) break;
+  for (int t = 0; t < NT; ++t)
 #pragma unroll
     for (int r = 0; r < NW; ++r) acc[r][t] = warp_sum(acc[r][t]);
-  }
+}
+
+template <typename T, int NW>
+__device__ __forceinline__ void shared_dots(const T* __restrict__ w, int64_t w_pitch, const T* __restrict__ x, int n, int nt, int lane, float (&acc)[NW][kShTok]) {
+  if (nt == 1) shared_dots_of<T, NW, 1>(w, w_pitch, x, n, nt, lane, acc);
+  else if (nt == 2) shared_dots_of<T, NW, 2>(w, w_pitch, x, n, nt, lane, acc);
+  else if (nt <= 4) shared_dots_of<T, NW, 4>(w, w_pitch, x, n, nt, lane, acc);
+  else shared_dots_of<T, NW, kShTok>(w, w_pitch, x, n, nt, lane, acc);
 }
 
 template <typename T>
@@ -332,14 +340,14 @@ __device__ __forceinline__ float as_dtype(float v) {   // v rounded to T
   return load_as_float(&r, 0);
 }
 
-template <typename T, bool GATED>
+template <typename T, bool GATED, bool SHARED>
 __global__ void __launch_bounds__(256) moe_gemv_up_kernel(const T* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ w_up,
                                                           T* __restrict__ hidden, int pairs, int top, int d, int ff, float limit, float alpha, SharedExpert sh) {
   griddep_launch();
   griddep_wait();
   const int p = blockIdx.y, lane = threadIdx.x & 31;
   const int f = blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (GATED && p >= pairs) {
+  if (SHARED && p >= pairs) {
     if (f >= sh.ff) return;
     const int t0 = (p - pairs) * kShTok, nt = min(kShTok, sh.tokens - t0);
     float acc[2][kShTok];
@@ -381,7 +389,7 @@ __global__ void __launch_bounds__(256) moe_gemv_up_kernel(const T* __restrict__ 
 }
 
 // decode: out[t, c] = sum_k wts[t, k] * T(W_down[ids[t, k]][c, :] . hidden[t * top + k, :]); one warp per c
-template <typename T>
+template <typename T, bool SHARED>
 __global__ void __launch_bounds__(256) moe_gemv_down_kernel(const T* __restrict__ hidden, const int* __restrict__ ids,
                                                             const float* __restrict__ wts, const T* __restrict__ w_down,
                                                             T* __restrict__ out, int tokens, int top, int d, int ff, SharedExpert sh) {
@@ -390,7 +398,7 @@ __global__ void __launch_bounds__(256) moe_gemv_down_kernel(const T* __restrict_
   const int t = blockIdx.y, lane = threadIdx.x & 31;
   const int c = blockIdx.x * 8 + (threadIdx.x >> 5);
   if (c >= d) return;
-  if (t >= tokens) {
+  if (SHARED && t >= tokens) {
     const int t0 = (t - tokens) * kShTok, nt = min(kShTok, sh.tokens - t0);
     float acc[1][kShTok];
     shared_dots<T, 1>(reinterpret_cast<const T*>(sh.down) + (int64_t)c * sh.ff, 0, reinterpret_cast<const T*>(sh.hidden) + (int64_t)t0 * sh.ff, sh.ff, nt, lane, acc);
@@ -508,14 +516,21 @@ int b200_moe_gemv(const void* x, const int32_t* ids, const float* weights, const
   const SharedExpert sh{shared_up, shared_down, shared_hidden, shared_out, shared_up ? shared_ff : 0, (int)tokens};
   const int pairs = (int)(tokens * top), extra = shared_up ? (int)((tokens + kShTok - 1) / kShTok) : 0, ffm = shared_ff > ff && shared_up ? shared_ff : ff;
   B200_FLOAT_TYPES(dtype, T, {
-    if (gated)
-      B200_CUDA(launch(moe_gemv_up_kernel<T, true>, dim3((unsigned)((ffm + 7) / 8), (unsigned)(pairs + extra)), dim3(256), 0, st, (const T*)x, ids,
+    if (shared_up)
+      B200_CUDA(launch(moe_gemv_up_kernel<T, true, true>, dim3((unsigned)((ffm + 7) / 8), (unsigned)(pairs + extra)), dim3(256), 0, st, (const T*)x, ids,
+                       (const T*)w_up, (T*)hidden, pairs, top, d, ff, limit, alpha, sh));
+    else if (gated)
+      B200_CUDA(launch(moe_gemv_up_kernel<T, true, false>, dim3((unsigned)((ff + 7) / 8), (unsigned)pairs), dim3(256), 0, st, (const T*)x, ids,
                        (const T*)w_up, (T*)hidden, pairs, top, d, ff, limit, alpha, sh));
     else
-      B200_CUDA(launch(moe_gemv_up_kernel<T, false>, dim3((unsigned)((ff + 7) / 8), (unsigned)pairs), dim3(256), 0, st, (const T*)x, ids,
+      B200_CUDA(launch(moe_gemv_up_kernel<T, false, false>, dim3((unsigned)((ff + 7) / 8), (unsigned)pairs), dim3(256), 0, st, (const T*)x, ids,
                        (const T*)w_up, (T*)hidden, pairs, top, d, ff, limit, alpha, sh));
-    B200_CUDA(launch(moe_gemv_down_kernel<T>, dim3((unsigned)((d + 7) / 8), (unsigned)(tokens + extra)), dim3(256), 0, st, (const T*)hidden, ids, weights,
-                     (const T*)w_down, (T*)out, (int)tokens, top, d, ff, sh));
+    if (shared_up)
+      B200_CUDA(launch(moe_gemv_down_kernel<T, true>, dim3((unsigned)((d + 7) / 8), (unsigned)(tokens + extra)), dim3(256), 0, st, (const T*)hidden, ids, weights,
+                       (const T*)w_down, (T*)out, (int)tokens, top, d, ff, sh));
+    else
+      B200_CUDA(launch(moe_gemv_down_kernel<T, false>, dim3((unsigned)((d + 7) / 8), (unsigned)tokens), dim3(256), 0, st, (const T*)hidden, ids, weights,
+                       (const T*)w_down, (T*)out, (int)tokens, top, d, ff, sh));
   });
   return B200_OK;
 }

@@ -17,8 +17,8 @@ those few; experts are gated with clamped branches, W_down (g sigmoid(alpha g) (
 
 ``SharedSparseExperts``: the `top` largest logits weighted by a softmax among them, plain gated experts W_down (silu(W_gate x) * (W_up x)),
 and a shared expert of that form times the sigmoid of one projected number per token.  The router's rows and that number's row are
-one weight: few tokens run them in the routing kernel, many as one matrix product with fp32 logits.  ``terms`` hands the parts of the
-result to the residual kernel, which weights and sums them (``K.gated_residual``).
+one weight and one matrix product with fp32 results.  ``terms`` hands the parts of the result to the residual kernel, which weights
+and sums them (``K.gated_residual``).
 """
 from __future__ import annotations
 
@@ -132,8 +132,6 @@ class ClampedSparseExperts(nn.Module):
 
 
 class SharedSparseExperts(nn.Module):
-    ROUTE_MM_MIN_ROWS = 32    # from this many tokens on the router's logits are one matrix product
-
     def __init__(self, width: int, spec: SharedMoESpec) -> None:
         super().__init__()
         self.spec = spec
@@ -149,7 +147,7 @@ class SharedSparseExperts(nn.Module):
     def route(self, x: torch.Tensor):
         """-> expert ids int32 (n, top), their weights fp32 (n, top), the shared expert's gate fp32 (n,) or None"""
         sp, shared = self.spec, self.shared_up is not None
-        if x.shape[0] >= self.ROUTE_MM_MIN_ROWS and sp.top <= 32 and sp.experts <= 3072:
+        if sp.top <= 32 and sp.experts <= 3072:
             res = K.moe_route_logits(K.mm_f32(x, self.w_route), sp.experts, sp.top, gate=shared)
         else:
             res = K.moe_route(x, self.w_route[: sp.experts], None, sp.top, 1, 1, topk_softmax=True, gate_w=self.w_route[sp.experts] if shared else None)

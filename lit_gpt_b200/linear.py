@@ -93,7 +93,7 @@ class DecayLinearAttention(nn.Module):
 class Retention(nn.Module):
     def __init__(self, width: int, spec: RetentionSpec, eps: float, projections: bool = True) -> None:
         """projections=False: the input and output projections belong to whoever runs this mixer beside another one (``parallel``), through
-        ``turned``, and ``read_out``."""
+        ``turned`` and ``read_out``."""
         super().__init__()
         self.spec, self.eps, self.width = spec, eps, width
         H, dk, dv = spec.heads, spec.dim, spec.vdim
